@@ -4,7 +4,8 @@
  * layer results, latent (compressed key/value) attention with a softmax sink and an output gate, clipped-GLU experts
  * with a softmax top-k router; residual kept as several streams, gated per-channel recurrences, attention over chunks
  * with a ring cache; post-norm residual, causal attention with a sink, matrix-state recurrences (decayed linear
- * attention, state-space duality), sigmoid routers with group-limited choice.  Every constant of a mechanism is a parameter.
+ * attention, state-space duality, gated delta rule), sigmoid routers with group-limited choice, latent attention under a
+ * sliding window.  Every constant of a mechanism is a parameter.
  *
  * Same boundary rules as ao_b200.h: device pointers + sizes + cudaStream_t as void*; nothing is allocated, freed,
  * synchronised or retained; every entry point can be captured into a CUDA graph; 0 = ok, else an AO_B200_ERR_* code.
@@ -421,6 +422,92 @@ AO_B200_API int ao_lm_router_topk_renorm_logits(const float* logits, int64_t ld,
 /* ao_lm_expert_gate_up for experts without a gate: y[p][ff] = act(w_up[e] h[t]); act 0: relu(.)^2. */
 AO_B200_API int ao_lm_expert_up_act(const void* h, const void* w_up, int dt, const int32_t* idx, int64_t n, int top, int64_t width,
                                     int64_t ff, int64_t expert_stride, int act, void* y, void* stream);
+
+/* ---------------------------------------------------------------------------------------------------------------
+ * Parallel sublayers on a pre-norm RMS residual (one input projection and one output product per layer: the row kernels
+ * below read and write parts of wider rows), gated delta rule, latent attention under a sliding window, values mixed with
+ * an earlier layer's, xIELU units.
+ */
+
+/* x[t][:] = table[tok[t]][:] * scale  (fp32 out) */
+AO_B200_API int ao_lm_embed_scaled(const void* table, int dt, const int64_t* tok, int64_t n, int64_t width, float scale, float* x,
+                                   void* stream);
+
+/* x[r] += y[r] (fp32 [n][width]; null: nothing is added);  out[i] = x[r] / sqrt(mean(x[r]^2) + eps) * weight in `dt` (weight
+ * null: no norm, only the add), r = rows ? rows[i] : i, i < m (rows only without y). */
+AO_B200_API int ao_lm_add_rms_norm(float* x, const float* y, const int32_t* rows, int64_t m, int64_t width, const void* weight, int dt,
+                                   float eps, void* out, void* stream);
+
+/* out[t][c] = pos * z^2 + z / 2 for z = in[t][c] > 0, neg * (exp(z) - 1 - z) + z / 2 otherwise; fp32 in, `dt` out, row strides. */
+AO_B200_API int ao_lm_xielu_rows(const float* in, int64_t ld, int64_t n, int64_t cols, float pos, float neg, void* out, int64_t ld_out,
+                                 int dt, void* stream);
+
+/* ao_lm_qkv_rotary_prep with a factor on cosine and sine (amp) and, with v_first (`dt` [n][v_width], another layer's values of
+ * the same rows), values (1 - v_mix) * v + v_mix * v_first. */
+AO_B200_API int ao_lm_qkv_rotary_mix_prep(const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off,
+                                          const void* q_bias, const void* k_bias, const void* v_bias, const int32_t* pos,
+                                          const float* inv_freq, int rot_dims, int pairing, float amp, const void* v_first,
+                                          float v_mix, int64_t n, int q_heads, int k_heads, int d, int v_width, int dt, float* qn,
+                                          void* kn, void* vn, void* stream);
+
+/* ao_lm_gated_group_norm with a row stride for the output and, shared_weight != 0, one weight of width / groups values for
+ * every group. */
+AO_B200_API int ao_lm_gated_group_norm_rows(const float* y, int64_t ldy, const float* gate, int64_t ldg, int mode, int64_t n,
+                                            int64_t width, int groups, const void* weight, int shared_weight, int dt, float eps,
+                                            void* out, int64_t ld_out, void* stream);
+
+/* Inputs of the gated delta rule from an fp32 projection row: the 2 G d + H dv channels [q | k | v] at conv_off through a
+ * causal convolution over time (conv_w: `dt` [taps][channels], last tap = the current row; earlier inputs from
+ * conv_state[slot][taps - 1][channels], zeros in front of position 0) and SiLU; q and k of every head divided by
+ * sqrt(sum of squares + unit_eps), q times q_scale -> qk [n][2][G][dp] (dp = d rounded up to 4, zeros beyond d), v [n][H dv];
+ * gb[t][h] = { exp(-exp(a_log) * softplus(proj[a_off + h] + dt_bias)), sigmoid(proj[b_off + h]) }.  All outputs fp32. */
+AO_B200_API int ao_lm_delta_prep(const float* proj, int64_t ld, int64_t conv_off, int64_t a_off, int64_t b_off, int64_t n, int H, int G,
+                                 int d, int dp, int dv, int taps, const void* conv_w, const float* conv_state, const int32_t* slot,
+                                 const int32_t* pos, const int32_t* back, const void* a_log, const void* dt_bias, int dt,
+                                 float unit_eps, float q_scale, float* qk, float* v, float* gb, void* stream);
+
+/* Gated delta rule per head (fp32 state[slots][H][dv][dp], zeros at position 0): S <- g S; u = beta (v - S^T k);
+ * S <- S + k u^T; out[t][h] = S^T q (fp32 [n][H dv]); head h reads group h / (H / G) of q and k.  seg_first / seg_count: the
+ * step's segments, whole.  block: tokens folded in at a time, 4 (segments of several rows) or 1; the same sums in another
+ * order.  With conv_x (fp32, row stride ld_conv), the last taps - 1 rows of every segment of its `channels` values become
+ * conv_state[slot] (the memory of the convolution that made q, k and v). */
+AO_B200_API int ao_lm_delta_recurrence(const float* qk, const float* v, const float* gb, int H, int G, int dp, int dv, float* state,
+                                       const int32_t* slot, const int32_t* pos, const int32_t* seg_first, const int32_t* seg_count,
+                                       int n_segments, int block, const float* conv_x, int64_t ld_conv, int64_t channels, int taps,
+                                       float* conv_state, float* out, void* stream);
+
+/* Projection row (fp32) -> cq[t] = RMS norm of the Rq values at q_off (weight q_norm), c[t] = RMS norm of the R values at
+ * kv_off (weight c_norm), kr[t] = the dr values behind them, rotated (pairs (2i, 2i+1), i < rot_dims / 2, angle
+ * pos * inv_freq[i], amp on cosine and sine).  All in `dt`. */
+AO_B200_API int ao_lm_latent_low_prep(const float* proj, int64_t ld, int64_t n, int64_t q_off, int Rq, int64_t kv_off, int R, int dr,
+                                      const void* q_norm, const void* c_norm, int dt, float eps, int rot_dims, const float* inv_freq,
+                                      float amp, const int32_t* pos, void* cq, void* c, void* kr, void* stream);
+/* q fp32 [n][H][dn + dr] -> qn[h][t][dn] in `dt`, qr[t][h][dr] rotated likewise, fp32. */
+AO_B200_API int ao_lm_latent_query_prep(const float* q, int64_t n, int H, int dn, int dr, int dt, int rot_dims, const float* inv_freq,
+                                        float amp, const int32_t* pos, void* qn, float* qr, void* stream);
+
+/* ao_lm_latent_attention under a sliding window: row t sees keys pos[t] - window + 1 .. pos[t] of its sequence.  Compressed
+ * rows of earlier steps come from a ring (position p in row p % ring, ring >= window), the step's own from c [n][R] /
+ * kr [n][dr] (back[t] = rows of the same segment in front of row t); ao_lm_ring_append stores them after the attention.
+ * sink and gate are optional (null).  The key splits cover window + tile_tokens - 1 keys. */
+AO_B200_API int ao_lm_window_latent_attention(const float* qa, const float* qr, const void* ring_c, const void* ring_kr, const void* c,
+                                              const void* kr, int dt, int ring, const int32_t* slot, const int32_t* pos,
+                                              const int32_t* back, const int32_t* tile_first, const int32_t* tile_count, int n_tiles,
+                                              int64_t n, int H, int R, int dr, float scale, int window, const void* sink,
+                                              const float* gate, int n_split, void* workspace, int64_t workspace_bytes, void* out,
+                                              void* stream);
+/* ao_lm_latent_attention_expanded under a sliding window, over rows that ao_lm_latent_rows_gather made contiguous: kx[row][h][dn]
+ * and vx[row][h][dv] with row strides ldk / ldv, kr[row][dr]; tile_kv_row[tile] = the row that key 0 of the tile's sequence
+ * would have (negative when its rows start at a later key).  sink and gate are optional. */
+AO_B200_API int ao_lm_window_latent_attention_expanded(const void* qn, const float* qr, const void* kx, int64_t ldk, const void* vx,
+                                                       int64_t ldv, const void* kr, int dt, const int32_t* pos,
+                                                       const int32_t* tile_first, const int32_t* tile_count,
+                                                       const int32_t* tile_kv_row, int n_tiles, int64_t n, int H, int dn, int dr,
+                                                       int dv, float scale, int window, const void* sink, const float* gate,
+                                                       void* out, int64_t ld_out, void* stream);
+/* out row i = row src[i] of c / kr when src[i] >= 0, else row -1 - src[i] of ring_c / ring_kr (slot * ring + position % ring). */
+AO_B200_API int ao_lm_latent_rows_gather(const int32_t* src, int64_t rows, const void* c, const void* kr, const void* ring_c,
+                                         const void* ring_kr, int dt, int R, int dr, void* out_c, void* out_kr, void* stream);
 
 #ifdef __cplusplus
 }

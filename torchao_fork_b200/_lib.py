@@ -208,6 +208,24 @@ LM_SIGNATURES = {
                                       _i32, _i32, _i32, _i32, _i32, _f32, _f32, _i32, _f32, _f32, _vp, _i64, _vp],
     "ao_lm_router_topk_renorm_logits": [_vp, _i64, _vp, _i64, _i32, _i32, _i32, _vp, _vp, _vp, _vp],
     "ao_lm_expert_up_act": [_vp, _vp, _i32, _vp, _i64, _i32, _i64, _i64, _i64, _i32, _vp, _vp],
+    "ao_lm_embed_scaled": [_vp, _i32, _vp, _i64, _i64, _f32, _vp, _vp],
+    "ao_lm_add_rms_norm": [_vp, _vp, _vp, _i64, _i64, _vp, _i32, _f32, _vp, _vp],
+    "ao_lm_xielu_rows": [_vp, _i64, _i64, _i64, _f32, _f32, _vp, _i64, _i32, _vp],
+    "ao_lm_qkv_rotary_mix_prep": [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _f32, _vp, _f32, _i64, _i32, _i32,
+                                  _i32, _i32, _i32, _vp, _vp, _vp, _vp],
+    "ao_lm_gated_group_norm_rows": [_vp, _i64, _vp, _i64, _i32, _i64, _i64, _i32, _vp, _i32, _i32, _f32, _vp, _i64, _vp],
+    "ao_lm_delta_prep": [_vp, _i64, _i64, _i64, _i64, _i64, _i32, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32,
+                         _f32, _f32, _vp, _vp, _vp, _vp],
+    "ao_lm_delta_recurrence": [_vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _vp, _i64, _i64, _i32, _vp,
+                               _vp, _vp],
+    "ao_lm_latent_low_prep": [_vp, _i64, _i64, _i64, _i32, _i64, _i32, _i32, _vp, _vp, _i32, _f32, _i32, _vp, _f32, _vp, _vp, _vp, _vp,
+                              _vp],
+    "ao_lm_latent_query_prep": [_vp, _i64, _i32, _i32, _i32, _i32, _i32, _vp, _f32, _vp, _vp, _vp, _vp],
+    "ao_lm_window_latent_attention": [_vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _i32, _i64, _i32, _i32, _i32,
+                                      _f32, _i32, _vp, _vp, _i32, _vp, _i64, _vp, _vp],
+    "ao_lm_window_latent_attention_expanded": [_vp, _vp, _vp, _i64, _vp, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i64, _i32, _i32,
+                                               _i32, _i32, _f32, _i32, _vp, _vp, _vp, _i64, _vp],
+    "ao_lm_latent_rows_gather": [_vp, _i64, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _vp, _vp, _vp],
 }
 _LM_RESTYPES = {"ao_lm_last_cuda_error": ctypes.c_char_p, "ao_lm_latent_attention_workspace_bytes": _i64, "ao_lm_scan_workspace_bytes": _i64, "ao_lm_outer_recurrence_workspace_bytes": _i64, "ao_lm_channel_recurrence_workspace_bytes": _i64, "ao_lm_window_attention_workspace_bytes": _i64,
                 "ao_lm_chunk_attention_workspace_bytes": _i64}

@@ -93,7 +93,8 @@ class SlotAllocator:
 
 class LatentKVCache(nn.Module):
     """What a latent-attention layer keeps per position instead of keys and values: the normed latent
-    `c` [slots][S][rank] and the rotated key part shared by all heads `kr` [slots][S][rot_dim]."""
+    `c` [slots][S][rank] and the rotated key part shared by all heads `kr` [slots][S][rot_dim].  Under a sliding window S is
+    a ring as long as the window (position p in row p % S); otherwise S is the longest sequence."""
 
     def __init__(self, n_slots, max_seq_length, rank, rot_dim, dtype=torch.bfloat16, device=None):
         super().__init__()

@@ -30,21 +30,9 @@ import torch.nn as nn
 
 from ..cache import MatrixState, SequenceStates, TokenShiftState, WindowKVCache
 from ..checkpoint import read_config, read_safetensors
+from ..rotary import RotaryArgs
 
 NO_WINDOW = 1 << 30     # a mask without a window size: plain causal attention
-
-
-@dataclass
-class RotaryArgs:
-    dims: int = 0               # 0: no rotation
-    base: float = 10000.0
-
-    def inv_freq(self, device) -> Optional[torch.Tensor]:
-        """base^(-2i/dims), i < dims/2, rounded once to fp32."""
-        if self.dims == 0:
-            return None
-        i = torch.arange(self.dims // 2, dtype=torch.float64)
-        return torch.pow(torch.tensor(self.base, dtype=torch.float64), -2.0 * i / self.dims).to(torch.float32).to(device)
 
 
 @dataclass
@@ -94,10 +82,10 @@ class LayerArgs:
 
 
 def _rot(m) -> RotaryArgs:
-    r = m.get("rot")
-    if not r:
-        return RotaryArgs()
-    return RotaryArgs(int(r["dims"]), float(r["base"]))
+    r = RotaryArgs.from_dict(m.get("rot"))
+    if r.scaling is not None:
+        raise NotImplementedError("Fedipel's rotations are not scaled")
+    return r
 
 
 @dataclass
@@ -175,7 +163,7 @@ class FedipelArgs:
         out = []
         for lay in self.layers:
             m, f = lay.mixer, lay.mlp
-            rot = {"base": m.rot.base, "dims": m.rot.dims} if lay.type != "wkv" and m.rot.dims else None
+            rot = m.rot.to_dict() if lay.type != "wkv" else None
             if lay.type == "retention":
                 mx = {"decay": list(m.decay), "dim": m.dim, "heads": m.heads, "vdim": m.vdim}
             elif lay.type == "wkv":

@@ -48,6 +48,9 @@ def _load_builtin():
     from .fedipel import model as _fedipel
     register(Family("fedipel", from_folder=_fedipel.Fedipel.from_checkpoint, from_name=_fedipel.Fedipel.from_name,
                     names=lambda: list(_fedipel.fedipel_configs)))
+    from .rigalorn import model as _rigalorn
+    register(Family("rigalorn", from_folder=_rigalorn.Rigalorn.from_checkpoint, from_name=_rigalorn.Rigalorn.from_name,
+                    names=lambda: list(_rigalorn.rigalorn_configs)))
 
 
 def architecture_of(folder) -> str:

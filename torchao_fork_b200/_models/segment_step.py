@@ -42,6 +42,7 @@ class StepMeta:
     attn: Dict[tuple, tuple]   # attention shape -> (tile_first, tile_count, n_tiles, tensor-core form?)
     seg: tuple           # (first row, rows, n) of the step's segments, whole
     rec: Optional[tuple] = None   # tiles of the matrix-state recurrences (as `scan`), when some segment is longer than one tile
+    extra: Dict[tuple, torch.Tensor] = {}   # a family's own int32 tables (`_piece_tables`)
 
 
 def segments_of(slot: np.ndarray, pos: np.ndarray):
@@ -120,6 +121,15 @@ class SegmentStepEngine:
         _lib.lm_check(self.L.ao_lm_chunk_attention_prompt_plan(self.dt, H, G, d, dv, ctypes.byref(pr)), "chunk_attention_prompt_plan")
         return tr.value, chunk, pr.value
 
+    def _prompt_form(self, shape, starts, counts, pos) -> bool:
+        """Whether a step that brings enough rows may attend with the tensor-core form for this shape (default: yes)."""
+        return True
+
+    def _piece_tables(self, starts, counts, slot, pos, forms, tiles) -> Dict[tuple, np.ndarray]:
+        """int32 tables that a family's own kernels need for a piece, sent along with the other metadata (meta.extra).
+        forms: attention shape -> (tile rows, span, tensor-core form?); tiles: that triple -> (first rows, row counts)."""
+        return {}
+
     # ------------------------------------------------------------------------------------------------ public
     @torch.no_grad()
     def step(self, segments: Sequence[Tuple[int, Union[torch.Tensor, Sequence[int]]]],
@@ -177,14 +187,16 @@ class SegmentStepEngine:
             parts += [seg0, segn]
         attn_np = {}
         prompt = n >= PROMPT_MIN_ROWS * len(starts)
-        meta_shapes = {shape: (self.prompt_keys[shape] if prompt and shape in self.prompt_keys else key)
-                       for shape, key in self.attn_keys.items()}
+        meta_shapes = {shape: (self.prompt_keys[shape] if prompt and shape in self.prompt_keys and self._prompt_form(shape, starts, counts, pos)
+                               else key) for shape, key in self.attn_keys.items()}
         for key in sorted(set(meta_shapes.values())):
             attn_np[key] = chunk_tiles(starts, counts, pos, key[0], key[1])
             parts += list(attn_np[key])
         rec = scan_tiles(starts, counts, REC_TILE) if getattr(self, "matrix_recurrences", False) else None
         if rec is not None and rec[2] is not None:
             parts += list(rec)
+        extra = self._piece_tables(starts, counts, slot, pos, meta_shapes, attn_np)
+        parts += list(extra.values())
         packed = torch.from_numpy(np.concatenate(parts)).to(self.dev, non_blocking=True)
         o = [0]
 
@@ -211,6 +223,7 @@ class SegmentStepEngine:
         meta.attn = {shape: tables[key] for shape, key in meta_shapes.items()}
         if rec is not None and rec[2] is not None:
             meta.rec = (take(len(rec[0])), take(len(rec[0])), len(rec[0]), take(len(rec[2])), take(len(rec[2])), len(rec[2]))
+        meta.extra = {name: take(len(t)) for name, t in extra.items()}
         return d_tok, meta
 
     def _run(self, tok: np.ndarray, slot: np.ndarray, pos: np.ndarray) -> torch.Tensor:

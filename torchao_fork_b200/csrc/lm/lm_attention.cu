@@ -22,6 +22,17 @@ __host__ __device__ inline int head_quads_per_cta(int H) {
   return q >= 8 ? 8 : q >= 4 ? 4 : q >= 2 ? 2 : 1;
 }
 
+constexpr int kNoWindow = 0x7fffffff;
+
+// What a sliding window adds to the kernels: a row at position i sees keys i - window + 1 .. i; the step's own rows are read
+// from c / kr (step rows in front of a row: back), earlier ones from the slot's ring.
+template <typename T>
+struct WindowArgs {
+  int window = kNoWindow;
+  const T *c = nullptr, *kr = nullptr;
+  const int32_t* back = nullptr;
+};
+
 constexpr int kPrefetch = 10;   // 16-byte chunks per thread held in registers for the next key tile
 
 // a 16-byte load that stays where it is written: the compiler may not sink it towards its first use
@@ -31,11 +42,27 @@ __device__ __forceinline__ uint4 ld16(const void* p) {
   return r;
 }
 
-// chunk `ch` of the cached row `key`: the first cr chunks are the latent, the rest the rotated key part
+// Where the compressed rows of one sequence lie: position p in row p % rows of its slot (a full cache never wraps, a window's
+// ring does); positions the step itself brings, from step0 on, in the step's own rows when there are any (step_c null: the
+// cache already holds them).
 template <typename T>
-__device__ __forceinline__ const T* chunk_src(const T* cbase, const T* kbase, int key, int ch, int cr, int R, int dr) {
+struct LatentRows {
+  const T *c, *kr, *step_c, *step_kr;
+  int rows, step0, R, dr;
+  __device__ __forceinline__ const T* latent(int key) const {
+    if (step_c && key >= step0) return step_c + (int64_t)(key - step0) * R;
+    return c + (int64_t)(key < rows ? key : key % rows) * R;
+  }
+  __device__ __forceinline__ const T* rotated(int key) const {
+    if (step_c && key >= step0) return step_kr + (int64_t)(key - step0) * dr;
+    return kr + (int64_t)(key < rows ? key : key % rows) * dr;
+  }
+};
+// chunk `ch` of the compressed row `key`: the first cr chunks are the latent, the rest the rotated key part
+template <typename T>
+__device__ __forceinline__ const T* chunk_src(const LatentRows<T>& src, int key, int ch, int cr) {
   constexpr int kPer = 16 / (int)sizeof(T);
-  return ch < cr ? cbase + (int64_t)key * R + ch * kPer : kbase + (int64_t)key * dr + (ch - cr) * kPer;
+  return ch < cr ? src.latent(key) + ch * kPer : src.rotated(key) + (ch - cr) * kPer;
 }
 // 16 bytes of a cached row -> fp32 in shared memory
 template <typename T>
@@ -55,16 +82,15 @@ __device__ __forceinline__ void store_chunk<float>(const uint4& u, float* dst) {
 }
 // all of a thread's loads for the tile that starts at key k0 are issued before any is used
 template <typename T>
-__device__ __forceinline__ void fetch_tile(uint4 (&pf)[kPrefetch], const T* cbase, const T* kbase, int k0, int k_hi, int cpk,
-                                           int cr, int R, int dr, int total_chunks) {
-  (void)cpk;
+__device__ __forceinline__ void fetch_tile(uint4 (&pf)[kPrefetch], const LatentRows<T>& src, int k0, int k_hi, int cr,
+                                           int total_chunks) {
 #pragma unroll
   for (int b = 0; b < kPrefetch; ++b) {
     const int i = threadIdx.x + b * kWarps * 32;
     pf[b] = make_uint4(0, 0, 0, 0);
     if (i < total_chunks) {
       const int j = i & (kKeys - 1), ch = i / kKeys;   // consecutive lanes: consecutive keys (odd row pitch: no bank conflicts)
-      if (k0 + j < k_hi) pf[b] = ld16(chunk_src(cbase, kbase, k0 + j, ch, cr, R, dr));
+      if (k0 + j < k_hi) pf[b] = ld16(chunk_src(src, k0 + j, ch, cr));
     }
   }
 }
@@ -81,6 +107,19 @@ __device__ __forceinline__ void store_tile(const uint4 (&pf)[kPrefetch], float* 
   }
 }
 
+template <typename T>
+__device__ __forceinline__ LatentRows<T> latent_rows(const T* c_cache, const T* kr_cache, int64_t seq, int64_t S, int R, int dr,
+                                                     const int32_t* pos, int first, const WindowArgs<T>& win) {
+  LatentRows<T> s{c_cache + seq * S * R, kr_cache + seq * S * dr, nullptr, nullptr, (int)S, 0, R, dr};
+  if (win.c) {
+    const int back0 = win.back[first];
+    s.step_c = win.c + (int64_t)(first - back0) * R;
+    s.step_kr = win.kr + (int64_t)(first - back0) * dr;
+    s.step0 = pos[first] - back0;
+  }
+  return s;
+}
+
 template <typename T, int RPL>
 __global__ void __launch_bounds__(kWarps * 32)
 latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, const T* __restrict__ c_cache,
@@ -88,7 +127,7 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
                    const int32_t* __restrict__ pos, const int32_t* __restrict__ tile_first,
                    const int32_t* __restrict__ tile_count, int64_t n, int H, int R, int dr, float scale, int HQ,
                    int tiles_per_split, int n_split, const T* __restrict__ sink, const float* __restrict__ gate,
-                   T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml) {
+                   T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, WindowArgs<T> win) {
   extern __shared__ float smem[];
   const int D = R + dr, DP = D + 1;
   float* qs = smem;                         // [kWarps][D][4]
@@ -105,9 +144,15 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
   const int64_t seq = slot[first];
   int max_pos = 0;
   for (int i = 0; i < count && i < TQ; ++i) max_pos = max(max_pos, pos[first + i]);
-  const int k_lo = blockIdx.z * tiles_per_split * kKeys;
+  const int k_lo = max(0, pos[first] - win.window + 1) + blockIdx.z * tiles_per_split * kKeys;
   const int k_hi = min(k_lo + tiles_per_split * kKeys, max_pos + 1);
-  if (k_lo >= k_hi) return;   // uniform over the CTA: nothing of this split is visible to any of its tokens
+  if (k_lo >= k_hi) {   // uniform over the CTA: nothing of this split is visible to any of its tokens
+    if (win.window != kNoWindow && n_split > 1 && active && lane < 4 && head0 + lane < H) {   // the merge reads every split
+      const int64_t at = (t * H + head0 + lane) * n_split + blockIdx.z;
+      part_ml[at * 2] = -INFINITY, part_ml[at * 2 + 1] = 0.f;
+    }
+    return;
+  }
 
   // the warp's four query rows, interleaved so that one 16-byte broadcast load feeds four score rows
   float* myq = qs + (size_t)warp * D * 4;
@@ -152,14 +197,14 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
 #pragma unroll
     for (int i = 0; i < RPL; ++i) o[r][i] = 0.f;
   }
-  const T* cbase = c_cache + seq * S * R;
-  const T* kbase = kr_cache + seq * S * dr;
+  const LatentRows<T> src = latent_rows(c_cache, kr_cache, seq, S, R, dr, pos, first, win);
   constexpr int kVecElems = 16 / (int)sizeof(T);
   const bool vec = R % kVecElems == 0 && dr % kVecElems == 0 && reinterpret_cast<uintptr_t>(c_cache) % 16 == 0 &&
-                   reinterpret_cast<uintptr_t>(kr_cache) % 16 == 0;
+                   reinterpret_cast<uintptr_t>(kr_cache) % 16 == 0 && reinterpret_cast<uintptr_t>(win.c) % 16 == 0 &&
+                   reinterpret_cast<uintptr_t>(win.kr) % 16 == 0;
   const int cr = R / kVecElems, cpk = cr + dr / kVecElems, total_chunks = kKeys * cpk;   // 16-byte chunks per row / tile
   uint4 pf[kPrefetch];
-  if (vec) fetch_tile<T>(pf, cbase, kbase, k_lo, k_hi, cpk, cr, R, dr, total_chunks);
+  if (vec) fetch_tile<T>(pf, src, k_lo, k_hi, cr, total_chunks);
   for (int k0 = k_lo; k0 < k_hi; k0 += kKeys) {
     __syncthreads();   // the previous tile is consumed (and myq is written, first time round)
     if (vec) {
@@ -168,7 +213,7 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
         for (int i = threadIdx.x + kPrefetch * kWarps * 32; i < total_chunks; i += kWarps * 32) {
           const int j = i & (kKeys - 1), ch = i / kKeys;
           uint4 v = make_uint4(0, 0, 0, 0);
-          if (k0 + j < k_hi) v = ld16(chunk_src(cbase, kbase, k0 + j, ch, cr, R, dr));
+          if (k0 + j < k_hi) v = ld16(chunk_src(src, k0 + j, ch, cr));
           store_chunk<T>(v, ks + (size_t)j * DP + ch * kVecElems);
         }
       }
@@ -177,8 +222,8 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
         const int key = k0 + j;
         float* dst = ks + (size_t)j * DP;
         if (key < k_hi) {
-          const T* c = cbase + (int64_t)key * R;
-          const T* kr = kbase + (int64_t)key * dr;
+          const T* c = src.latent(key);
+          const T* kr = src.rotated(key);
           for (int d = lane; d < R; d += 32) dst[d] = ldf(c + d);
           for (int d = lane; d < dr; d += 32) dst[R + d] = ldf(kr + d);
         } else {
@@ -188,8 +233,8 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
     }
     __syncthreads();
     // the next tile's rows travel while this one is computed (registers are the second buffer)
-    if (vec && k0 + kKeys < k_hi) fetch_tile<T>(pf, cbase, kbase, k0 + kKeys, k_hi, cpk, cr, R, dr, total_chunks);
-    if (!active || k0 > my_pos) continue;   // uniform over the warp
+    if (vec && k0 + kKeys < k_hi) fetch_tile<T>(pf, src, k0 + kKeys, k_hi, cr, total_chunks);
+    if (!active || k0 > my_pos || k0 + kKeys <= my_pos - win.window + 1) continue;   // uniform over the warp
     float s[4] = {0.f, 0.f, 0.f, 0.f};
     const float* kk = ks + (size_t)lane * DP;
     const float4* q4 = reinterpret_cast<const float4*>(myq);
@@ -203,13 +248,13 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
       s[3] = fmaf(q.w, kv, s[3]);
     }
     const int key = k0 + lane;
-    const bool seen = key < k_hi && key <= my_pos;
+    const bool seen = key < k_hi && key <= my_pos && my_pos - key < win.window;
     float p[4];
 #pragma unroll
     for (int r = 0; r < 4; ++r) {
       const float sc = seen ? s[r] * scale : -INFINITY;
-      const float mn = fmaxf(m[r], warp_max(sc));   // finite: key k0 <= my_pos is seen
-      const float corr = __expf(m[r] - mn);         // exp(-inf) = 0 on the first tile
+      const float mn = fmaxf(m[r], warp_max(sc));   // -inf: the row has seen no key so far (a window that starts later)
+      const float corr = mn == -INFINITY ? 1.f : __expf(m[r] - mn);   // exp(-inf) = 0 on the first tile
       p[r] = seen ? __expf(sc - mn) : 0.f;
       m[r] = mn;
       l[r] = fmaf(l[r], corr, p[r]);
@@ -239,10 +284,10 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
     if (h >= H) break;
     const float lsum = warp_sum(l[r]);
     if (n_split == 1) {
-      const float sk = ldf(sink + h);
+      const float sk = sink ? ldf(sink + h) : -INFINITY;
       const float top = fmaxf(m[r], sk);
       const float e = __expf(m[r] - top);
-      const float k = gate[t * H + h] * e / (lsum * e + __expf(sk - top));
+      const float k = (gate ? gate[t * H + h] : 1.f) * e / (lsum * e + __expf(sk - top));
       T* dst = out + (t * H + h) * R;
 #pragma unroll
       for (int i = 0; i < RPL; ++i) {
@@ -290,7 +335,7 @@ latent_attn_mma_kernel(const float* __restrict__ qa, const float* __restrict__ q
                        const int32_t* __restrict__ tile_count, int64_t n, int H, int dr, float scale, int HB,
                        int tiles_per_split, int n_split, const __nv_bfloat16* __restrict__ sink,
                        const float* __restrict__ gate, __nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
-                       float* __restrict__ part_ml) {
+                       float* __restrict__ part_ml, WindowArgs<__nv_bfloat16> win) {
   using T = __nv_bfloat16;
   constexpr int R = 64 * NT;
   extern __shared__ float smem[];
@@ -307,18 +352,24 @@ latent_attn_mma_kernel(const float* __restrict__ qa, const float* __restrict__ q
   const int64_t seq = slot[first];
   int max_pos = 0;
   for (int i = 0; i < count; ++i) max_pos = max(max_pos, pos[first + i]);
-  const int k_lo = blockIdx.z * tiles_per_split * kKeys;
+  const int k_lo = max(0, pos[first] - win.window + 1) + blockIdx.z * tiles_per_split * kKeys;
   const int k_hi = min(k_lo + tiles_per_split * kKeys, max_pos + 1);
-  if (k_lo >= k_hi) return;
+  if (k_lo >= k_hi) {
+    const int r = threadIdx.x, tq = r / HB, h = head_base + r - tq * HB;
+    if (win.window != kNoWindow && n_split > 1 && r < kMmaRows && tq < count && h < H) {   // the merge reads every split
+      const int64_t at = ((int64_t)(first + tq) * H + h) * n_split + blockIdx.z;
+      part_ml[at * 2] = -INFINITY, part_ml[at * 2 + 1] = 0.f;
+    }
+    return;
+  }
   if (threadIdx.x < kMmaRows) {
     const int r = threadIdx.x, tq = r / HB, hh = r - tq * HB;
     row_pos[r] = (tq < count && head_base + hh < H) ? pos[first + tq] : -1;
   }
-  const T* cbase = c_cache + seq * S * R;
-  const T* kbase = kr_cache + seq * S * dr;
+  const LatentRows<T> src = latent_rows(c_cache, kr_cache, seq, S, R, dr, pos, first, win);
   const int cr = R / 8, cpk = cr + dr / 8, total_chunks = kKeys * cpk;
   uint4 pf[kPrefetch];
-  fetch_tile<T>(pf, cbase, kbase, k_lo, k_hi, cpk, cr, R, dr, total_chunks);
+  fetch_tile<T>(pf, src, k_lo, k_hi, cr, total_chunks);
   // queries of the 16 rows, split into TF32 high and low parts; 16-byte loads, four in flight per thread
   {
     const int cq = D / 4, total_q = kMmaRows * cq;
@@ -366,11 +417,11 @@ latent_attn_mma_kernel(const float* __restrict__ qa, const float* __restrict__ q
     for (int i = threadIdx.x + kPrefetch * kWarps * 32; i < total_chunks; i += kWarps * 32) {
       const int j = i & (kKeys - 1), ch = i / kKeys;
       uint4 v = make_uint4(0, 0, 0, 0);
-      if (k0 + j < k_hi) v = ld16(chunk_src(cbase, kbase, k0 + j, ch, cr, R, dr));
+      if (k0 + j < k_hi) v = ld16(chunk_src(src, k0 + j, ch, cr));
       store_chunk<T>(v, ks + (size_t)j * DP + ch * 8);
     }
     __syncthreads();
-    if (k0 + kKeys < k_hi) fetch_tile<T>(pf, cbase, kbase, k0 + kKeys, k_hi, cpk, cr, R, dr, total_chunks);
+    if (k0 + kKeys < k_hi) fetch_tile<T>(pf, src, k0 + kKeys, k_hi, cr, total_chunks);
     {   // scores: rows 16 x keys [8 nt_s, +8) over coordinates [8 kbeg, 8 kend)
       float acc[4] = {0.f, 0.f, 0.f, 0.f};
       const float* kb = ks + (size_t)(nt_s * 8 + g) * DP + tq4;
@@ -403,8 +454,8 @@ latent_attn_mma_kernel(const float* __restrict__ qa, const float* __restrict__ q
       const int kc = (i >> 1) * 8 + tq4 + (i & 1) * 4, key = k0 + kc;
       const float v0 = (sp[g * 33 + kc] + sp[kMmaRows * 33 + g * 33 + kc]) * scale;
       const float v1 = (sp[(g + 8) * 33 + kc] + sp[kMmaRows * 33 + (g + 8) * 33 + kc]) * scale;
-      s0[i] = (key < k_hi && key <= p0) ? v0 : -INFINITY;
-      s1[i] = (key < k_hi && key <= p1) ? v1 : -INFINITY;
+      s0[i] = (key < k_hi && key <= p0 && p0 - key < win.window) ? v0 : -INFINITY;
+      s1[i] = (key < k_hi && key <= p1 && p1 - key < win.window) ? v1 : -INFINITY;
       mx0 = fmaxf(mx0, s0[i]);
       mx1 = fmaxf(mx1, s1[i]);
     }
@@ -454,10 +505,10 @@ latent_attn_mma_kernel(const float* __restrict__ qa, const float* __restrict__ q
     const int64_t t = first + tq;
     const float mr = half ? m1 : m0, lr = half ? l1 : l0;
     if (n_split == 1) {
-      const float sk = __bfloat162float(sink[h]);
+      const float sk = sink ? __bfloat162float(sink[h]) : -INFINITY;
       const float top = fmaxf(mr, sk);
       const float e = __expf(mr - top);
-      const float k = gate[t * H + h] * e / (lr * e + __expf(sk - top));
+      const float k = (gate ? gate[t * H + h] : 1.f) * e / (lr * e + __expf(sk - top));
       T* dst = out + (t * H + h) * R + col0 + 2 * tq4;
 #pragma unroll
       for (int i = 0; i < NT; ++i)
@@ -481,16 +532,17 @@ __host__ __device__ inline bool mma_path(int dt, int H, int R, int dr) {
 template <typename T>
 __global__ void latent_attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          const int32_t* __restrict__ pos, int H, int R, int tiles_per_split, int n_split,
-                                         const T* __restrict__ sink, const float* __restrict__ gate, T* __restrict__ out) {
+                                         const T* __restrict__ sink, const float* __restrict__ gate, T* __restrict__ out,
+                                         int window) {
   __shared__ float wsplit[64];   // n_split <= 64: exp(m_s - top) / denominator, gate folded in
-  __shared__ float red[2];
   const int64_t row = blockIdx.x;
   const int64_t t = row / H;
   const int h = (int)(row - t * H);
-  const int ns = min(n_split, pos[t] / (tiles_per_split * kKeys) + 1);
+  // the splits that may hold keys of this row (under a window every split left its statistics)
+  const int ns = window != kNoWindow ? n_split : min(n_split, pos[t] / (tiles_per_split * kKeys) + 1);
   if (threadIdx.x < 32) {
     const int lane = threadIdx.x;
-    const float sk = ldf(sink + h);
+    const float sk = sink ? ldf(sink + h) : -INFINITY;
     float m_a = lane < ns ? part_ml[(row * n_split + lane) * 2] : -INFINITY;
     float m_b = lane + 32 < ns ? part_ml[(row * n_split + lane + 32) * 2] : -INFINITY;
     const float top = fmaxf(warp_max(fmaxf(m_a, m_b)), sk);
@@ -498,10 +550,9 @@ __global__ void latent_attn_merge_kernel(const float* __restrict__ part_o, const
     float den = (lane < ns ? part_ml[(row * n_split + lane) * 2 + 1] * e_a : 0.f) +
                 (lane + 32 < ns ? part_ml[(row * n_split + lane + 32) * 2 + 1] * e_b : 0.f);
     den = warp_sum(den) + __expf(sk - top);
-    const float k = gate[row] / den;
+    const float k = (gate ? gate[row] : 1.f) / den;
     wsplit[lane] = e_a * k;
     wsplit[lane + 32] = e_b * k;
-    (void)red;
   }
   __syncthreads();
   // blockIdx.y: which 128 output coordinates (one per thread), so that a decoded token's few rows still fill many SMs
@@ -509,16 +560,26 @@ __global__ void latent_attn_merge_kernel(const float* __restrict__ part_o, const
   if (d < R) {
     float acc = 0.f;
 #pragma unroll 8
-    for (int s = 0; s < ns; ++s) acc = fmaf(part_o[(row * n_split + s) * R + d], wsplit[s], acc);
+    for (int s = 0; s < ns; ++s) {
+      const float w = wsplit[s];     // 0: a split that saw no key may have left no sums
+      acc = w != 0.f ? fmaf(part_o[(row * n_split + s) * R + d], w, acc) : acc;
+    }
     stf(out + row * R + d, acc);
   }
+}
+
+// 32-key tiles that a row tile of `tile_tokens` tokens can see: keys 0 .. max_pos, or a window's worth of them
+inline int key_tiles(int max_pos, int window, int tile_tokens) {
+  int64_t keys = (int64_t)max_pos + 1;
+  if (window != kNoWindow) keys = (int64_t)window + tile_tokens - 1;
+  return (int)((keys + kKeys - 1) / kKeys);
 }
 
 template <typename T, int RPL>
 int launch(const float* qa, const float* qr, const void* c_cache, const void* kr_cache, int64_t S, const int32_t* slot,
            const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count, int n_tiles, int64_t n, int H, int R,
            int dr, float scale, const void* sink, const float* gate, int max_pos, int n_split, float* part_o,
-           float* part_ml, void* out, cudaStream_t st) {
+           float* part_ml, void* out, const WindowArgs<T>& win, cudaStream_t st) {
   const int HQ = head_quads_per_cta(H);
   const int D = R + dr;
   const size_t smem = ((size_t)kWarps * D * 4 + (size_t)kKeys * (D + 1)) * sizeof(float);
@@ -531,16 +592,16 @@ int launch(const float* qa, const float* qr, const void* c_cache, const void* kr
       set = true;
     }
   }
-  const int tiles = (max_pos + kKeys) / kKeys;                 // 32-key tiles that hold keys 0 .. max_pos
+  const int tiles = key_tiles(max_pos, win.window, kWarps / HQ);
   const int tps = (tiles + n_split - 1) / n_split;
   const int quads = (H + 3) / 4;
   dim3 grid((unsigned)n_tiles, (unsigned)((quads + HQ - 1) / HQ), (unsigned)n_split);
   kern<<<grid, kWarps * 32, smem, st>>>(qa, qr, static_cast<const T*>(c_cache), static_cast<const T*>(kr_cache), S, slot, pos,
                                         tile_first, tile_count, n, H, R, dr, scale, HQ, tps, n_split,
-                                        static_cast<const T*>(sink), gate, static_cast<T*>(out), part_o, part_ml);
+                                        static_cast<const T*>(sink), gate, static_cast<T*>(out), part_o, part_ml, win);
   if (n_split > 1)
     latent_attn_merge_kernel<T><<<dim3((unsigned)(n * H), (unsigned)((R + 127) / 128)), 128, 0, st>>>(part_o, part_ml, pos, H, R, tps, n_split,
-                                                                  static_cast<const T*>(sink), gate, static_cast<T*>(out));
+                                                                  static_cast<const T*>(sink), gate, static_cast<T*>(out), win.window);
   return lm_launch_status();
 }
 
@@ -548,7 +609,7 @@ template <int NT>
 int launch_mma(const float* qa, const float* qr, const void* c_cache, const void* kr_cache, int64_t S, const int32_t* slot,
                const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count, int n_tiles, int64_t n, int H, int dr,
                float scale, const void* sink, const float* gate, int max_pos, int n_split, float* part_o, float* part_ml,
-               void* out, cudaStream_t st) {
+               void* out, const WindowArgs<__nv_bfloat16>& win, cudaStream_t st) {
   using T = __nv_bfloat16;
   constexpr int R = 64 * NT;
   const int DP = R + dr + 4;
@@ -563,15 +624,15 @@ int launch_mma(const float* qa, const float* qr, const void* c_cache, const void
     }
   }
   const int HB = H < kMmaRows ? H : kMmaRows;
-  const int tiles = (max_pos + kKeys) / kKeys;
+  const int tiles = key_tiles(max_pos, win.window, kMmaRows / HB);
   const int tps = (tiles + n_split - 1) / n_split;
   dim3 grid((unsigned)n_tiles, (unsigned)((H + HB - 1) / HB), (unsigned)n_split);
   kern<<<grid, kWarps * 32, smem, st>>>(qa, qr, static_cast<const T*>(c_cache), static_cast<const T*>(kr_cache), S, slot, pos,
                                         tile_first, tile_count, n, H, dr, scale, HB, tps, n_split, static_cast<const T*>(sink),
-                                        gate, static_cast<T*>(out), part_o, part_ml);
+                                        gate, static_cast<T*>(out), part_o, part_ml, win);
   if (n_split > 1)
     latent_attn_merge_kernel<T><<<dim3((unsigned)(n * H), (unsigned)((R + 127) / 128)), 128, 0, st>>>(part_o, part_ml, pos, H, R, tps, n_split,
-                                                                  static_cast<const T*>(sink), gate, static_cast<T*>(out));
+                                                                  static_cast<const T*>(sink), gate, static_cast<T*>(out), win.window);
   return lm_launch_status();
 }
 
@@ -588,13 +649,12 @@ extern "C" int64_t ao_lm_latent_attention_workspace_bytes(int64_t n, int H, int 
   return n * H * n_split * (int64_t)(R + 2) * 4;
 }
 
-extern "C" int ao_lm_latent_attention(const float* qa, const float* qr, const void* c_cache, const void* kr_cache, int dt,
-                                      int64_t S, const int32_t* slot, const int32_t* pos, const int32_t* tile_first,
-                                      const int32_t* tile_count, int n_tiles, int64_t n, int H, int R, int dr, float scale,
-                                      const void* sink, const float* gate, int max_pos, int n_split, void* workspace,
-                                      int64_t workspace_bytes, void* out, void* stream) {
-  LM_CHECK_ARG(qa && qr && c_cache && kr_cache && slot && pos && tile_first && tile_count && sink && gate && out);
-  LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && R > 0 && dr >= 0 && S > 0 && max_pos >= 0 && max_pos < S && n_split >= 1 && n_split <= 64);
+template <typename T>
+static int dispatch_latent(const float* qa, const float* qr, const void* c_cache, const void* kr_cache, int dt, int64_t S,
+                           const int32_t* slot, const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count,
+                           int n_tiles, int64_t n, int H, int R, int dr, float scale, const void* sink, const float* gate,
+                           int max_pos, int n_split, void* workspace, int64_t workspace_bytes, void* out, const WindowArgs<T>& win,
+                           cudaStream_t st) {
   if (R > 512) return AO_B200_ERR_UNSUPPORTED;
   float *part_o = nullptr, *part_ml = nullptr;
   if (n_split > 1) {
@@ -602,25 +662,54 @@ extern "C" int ao_lm_latent_attention(const float* qa, const float* qr, const vo
     part_o = static_cast<float*>(workspace);
     part_ml = part_o + n * H * n_split * (int64_t)R;
   }
-  const cudaStream_t st = lm_stream(stream);
-  if (mma_path(dt, H, R, dr)) {
-#define LM_MMA(NT)                                                                                                            \
-  case NT:                                                                                                                    \
-    return launch_mma<NT>(qa, qr, c_cache, kr_cache, S, slot, pos, tile_first, tile_count, n_tiles, n, H, dr, scale, sink, gate, \
-                          max_pos, n_split, part_o, part_ml, out, st);
-    switch (R / 64) {
-      LM_MMA(1) LM_MMA(2) LM_MMA(3) LM_MMA(4) LM_MMA(5) LM_MMA(6) LM_MMA(7) LM_MMA(8)
-    }
+#define LM_ARGS qa, qr, c_cache, kr_cache, S, slot, pos, tile_first, tile_count, n_tiles, n, H
+#define LM_TAIL dr, scale, sink, gate, max_pos, n_split, part_o, part_ml, out, win, st
+  if constexpr (sizeof(T) == 2) {
+    if (mma_path(dt, H, R, dr)) {
+#define LM_MMA(NT) \
+  case NT:         \
+    return launch_mma<NT>(LM_ARGS, LM_TAIL);
+      switch (R / 64) {
+        LM_MMA(1) LM_MMA(2) LM_MMA(3) LM_MMA(4) LM_MMA(5) LM_MMA(6) LM_MMA(7) LM_MMA(8)
+      }
 #undef LM_MMA
+    }
   }
-#define LM_ATTN(RPL)                                                                                                        \
-  LM_DISPATCH(dt, return (launch<T, RPL>(qa, qr, c_cache, kr_cache, S, slot, pos, tile_first, tile_count, n_tiles, n, H, R, dr, \
-                                         scale, sink, gate, max_pos, n_split, part_o, part_ml, out, st)))
-  if (R <= 32) LM_ATTN(1);
-  else if (R <= 64) LM_ATTN(2);
-  else if (R <= 128) LM_ATTN(4);
-  else if (R <= 256) LM_ATTN(8);
-  else LM_ATTN(16);
-#undef LM_ATTN
+  if (R <= 32) return launch<T, 1>(LM_ARGS, R, LM_TAIL);
+  if (R <= 64) return launch<T, 2>(LM_ARGS, R, LM_TAIL);
+  if (R <= 128) return launch<T, 4>(LM_ARGS, R, LM_TAIL);
+  if (R <= 256) return launch<T, 8>(LM_ARGS, R, LM_TAIL);
+  return launch<T, 16>(LM_ARGS, R, LM_TAIL);
+#undef LM_ARGS
+#undef LM_TAIL
+}
+
+extern "C" int ao_lm_latent_attention(const float* qa, const float* qr, const void* c_cache, const void* kr_cache, int dt,
+                                      int64_t S, const int32_t* slot, const int32_t* pos, const int32_t* tile_first,
+                                      const int32_t* tile_count, int n_tiles, int64_t n, int H, int R, int dr, float scale,
+                                      const void* sink, const float* gate, int max_pos, int n_split, void* workspace,
+                                      int64_t workspace_bytes, void* out, void* stream) {
+  LM_CHECK_ARG(qa && qr && c_cache && kr_cache && slot && pos && tile_first && tile_count && sink && gate && out);
+  LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && R > 0 && dr >= 0 && S > 0 && max_pos >= 0 && max_pos < S && n_split >= 1 && n_split <= 64);
+  LM_DISPATCH(dt, return dispatch_latent<T>(qa, qr, c_cache, kr_cache, dt, S, slot, pos, tile_first, tile_count, n_tiles, n, H, R, dr,
+                                            scale, sink, gate, max_pos, n_split, workspace, workspace_bytes, out, WindowArgs<T>{},
+                                            lm_stream(stream)));
+  return AO_B200_OK;
+}
+
+extern "C" int ao_lm_window_latent_attention(const float* qa, const float* qr, const void* ring_c, const void* ring_kr, const void* c,
+                                             const void* kr, int dt, int ring, const int32_t* slot, const int32_t* pos,
+                                             const int32_t* back, const int32_t* tile_first, const int32_t* tile_count, int n_tiles,
+                                             int64_t n, int H, int R, int dr, float scale, int window, const void* sink,
+                                             const float* gate, int n_split, void* workspace, int64_t workspace_bytes, void* out,
+                                             void* stream) {
+  LM_CHECK_ARG(qa && (qr || dr == 0) && ring_c && (ring_kr || dr == 0) && c && (kr || dr == 0) && slot && pos && back && tile_first && tile_count && out);
+  LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && R > 0 && dr >= 0 && window > 0 && window < kNoWindow && ring >= window && n_split >= 1 && n_split <= 64);
+  LM_DISPATCH(dt, {
+    WindowArgs<T> win;
+    win.window = window, win.c = static_cast<const T*>(c), win.kr = static_cast<const T*>(kr), win.back = back;
+    return dispatch_latent<T>(qa, qr, ring_c, ring_kr, dt, ring, slot, pos, tile_first, tile_count, n_tiles, n, H, R, dr, scale, sink,
+                              gate, 0, n_split, workspace, workspace_bytes, out, win, lm_stream(stream));
+  });
   return AO_B200_OK;
 }

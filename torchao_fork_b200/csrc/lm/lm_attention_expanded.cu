@@ -11,7 +11,7 @@
 //   sink, gate, normalisation in fp32.
 // One CTA = 64 consecutive tokens of one sequence x one head (4 warps x 16 rows).  K and V tiles arrive by cp.async in
 // separate groups: the next keys load while the weights meet the values, the next values during the score product.
-#include "lm_common.cuh"
+#include "lm_mma.cuh"
 
 using namespace lm;
 
@@ -22,43 +22,6 @@ constexpr int kPN = 64;      // keys per tile
 constexpr int kPWarps = 4;
 constexpr int kPad = 8;      // bf16 elements added to every shared-memory row: 16-byte rows land on distinct banks
 
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
-  const uint32_t s = (uint32_t)__cvta_generic_to_shared(smem);
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
-  const uint32_t s = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(s));
-}
-__device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], const void* p) {
-  const uint32_t s = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(s));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-// x -> (bf16 part, what is left of x); the remainder is exact in fp32
-__device__ __forceinline__ float split_bf16(float& x) {
-  const float h = __bfloat162float(__float2bfloat16_rn(x));
-  x -= h;
-  return h;
-}
-
 template <int NV>   // value size = 16 NV
 __global__ void __launch_bounds__(kPWarps * 32)
 latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* __restrict__ qr,
@@ -67,7 +30,8 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
                             const int32_t* __restrict__ pos, const int32_t* __restrict__ tile_first,
                             const int32_t* __restrict__ tile_count, const int32_t* __restrict__ tile_kv_row, int64_t n, int H,
                             int dn, int dr, float scale, const __nv_bfloat16* __restrict__ sink,
-                            const float* __restrict__ gate, __nv_bfloat16* __restrict__ out) {
+                            const float* __restrict__ gate, __nv_bfloat16* __restrict__ out, int64_t ldk, int64_t ldv, int window,
+                            int64_t ld_out) {
   using T = __nv_bfloat16;
   constexpr int DV = 16 * NV;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -79,13 +43,13 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
   const int h = blockIdx.y;
   const int tile = gridDim.x - 1 - blockIdx.x;   // a prompt's last tiles see the most keys: they start first
   const int first = tile_first[tile], count = min(tile_count[tile], kPM);
-  const int64_t seq = slot[first];
-  const int64_t row0 = tile_kv_row[tile];
+  const int64_t row0 = tile_kv_row[tile];        // the row of key 0 (negative when a window's rows start at a later key)
   const int pos0 = pos[first];
   const int k_hi = pos[first + count - 1] + 1;   // keys 0 .. the last row's position
-  const T* kbase = kx + row0 * (int64_t)H * dn + (int64_t)h * dn;
-  const T* vbase = vx + row0 * (int64_t)H * DV + (int64_t)h * DV;
-  const T* rbase = kr_cache + seq * S * dr;
+  const int k_lo = max(0, pos0 - window + 1);    // the oldest key of the first row's window
+  const T* kbase = kx + row0 * ldk + (int64_t)h * dn;
+  const T* vbase = vx + row0 * ldv + (int64_t)h * DV;
+  const T* rbase = kr_cache + (slot ? slot[first] * S : row0) * dr;
   const int kc_n = dn / 8, kc = kc_n + dr / 8;   // 16-byte chunks of a key row
   constexpr int vc = DV / 8;
 
@@ -94,7 +58,7 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
       const int j = i / kc, c = i - j * kc, key = k0 + j;
       T* dst = Ks + (size_t)j * KP + c * 8;
       if (key < k_hi)
-        cp_async16(dst, c < kc_n ? kbase + (int64_t)key * H * dn + c * 8 : rbase + (int64_t)key * dr + (c - kc_n) * 8);
+        cp_async16(dst, c < kc_n ? kbase + key * ldk + c * 8 : rbase + (int64_t)key * dr + (c - kc_n) * 8);
       else
         *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
     }
@@ -104,14 +68,14 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
       const int j = i / vc, c = i - j * vc, key = k0 + j;
       T* dst = Vs + (size_t)j * VP + c * 8;
       if (key < k_hi)
-        cp_async16(dst, vbase + (int64_t)key * H * DV + c * 8);
+        cp_async16(dst, vbase + key * ldv + c * 8);
       else
         *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
     }
   };
-  load_k(0);
+  load_k(k_lo);
   cp_async_commit();
-  load_v(0);
+  load_v(k_lo);
   cp_async_commit();
   // the query tile (rows past the run are zero)
   for (int i = threadIdx.x; i < kPM * kc_n; i += kPWarps * 32) {
@@ -142,17 +106,17 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
   const T* kb_ptr = Ks + (size_t)((lane & 7) + (lane >> 4) * 8) * KP + ((lane >> 3) & 1) * 8;
   const T* vb_ptr = Vs + (size_t)((lane & 7) + ((lane >> 3) & 1) * 8) * VP + (lane >> 4) * 8;
   const int ks_main = DK / 16, ks_lo = dr / 16, ks_n = dn / 16;
-  // a warp whose rows all come before a key tile skips the tile (its weights there are all zero)
+  // a warp skips a key tile that lies wholly in its rows' future, or wholly behind the window of its first row
   const int warp_last = min(count, warp * 16 + 16) - 1;             // < warp * 16: the warp has no rows
   const int warp_hi = warp_last >= warp * 16 ? pos0 + warp_last + 1 : 0;
 
-  for (int k0 = 0; k0 < k_hi; k0 += kPN) {
+  for (int k0 = k_lo; k0 < k_hi; k0 += kPN) {
     cp_async_wait<1>();
     __syncthreads();   // keys of this tile (and, the first time, the queries) are in shared memory
     float s[kPN / 8][4];
 #pragma unroll
     for (int i = 0; i < kPN / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-    const bool live = k0 < warp_hi;
+    const bool live = k0 < warp_hi && k0 + kPN > pos0 + warp * 16 - window + 1;
     if (live) {
       for (int kk = 0; kk < ks_main + ks_lo; ++kk) {
         uint32_t a[4];
@@ -173,8 +137,8 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int key = k0 + i * 8 + 2 * t4 + e;
-        s[i][e] = key <= p0 ? s[i][e] * scale : -INFINITY;
-        s[i][2 + e] = key <= p1 ? s[i][2 + e] * scale : -INFINITY;
+        s[i][e] = key <= p0 && p0 - key < window ? s[i][e] * scale : -INFINITY;
+        s[i][2 + e] = key <= p1 && p1 - key < window ? s[i][2 + e] * scale : -INFINITY;
         mx0 = fmaxf(mx0, s[i][e]);
         mx1 = fmaxf(mx1, s[i][2 + e]);
       }
@@ -251,7 +215,8 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  const float sk = __bfloat162float(sink[h]);
+  const float sk = sink ? __bfloat162float(sink[h]) : -INFINITY;
+  const bool pairs = ld_out % 2 == 0;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int r = half ? r1 : r0;
@@ -260,11 +225,18 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
     const float mr = half ? m1 : m0, lr = half ? l1 : l0;
     const float top = fmaxf(mr, sk);
     const float e = __expf(mr - top);
-    const float k = gate[t * H + h] * e / (lr * e + __expf(sk - top));
-    T* dst = out + (t * H + h) * DV + 2 * t4;
+    const float k = (gate ? gate[t * H + h] : 1.f) * e / (lr * e + __expf(sk - top));
+    T* dst = out + t * ld_out + (int64_t)h * DV + 2 * t4;
 #pragma unroll
-    for (int i = 0; i < 2 * NV; ++i)
-      *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(o[i][2 * half] * k, o[i][2 * half + 1] * k);
+    for (int i = 0; i < 2 * NV; ++i) {
+      const float y0 = o[i][2 * half] * k, y1 = o[i][2 * half + 1] * k;
+      if (pairs) {
+        *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(y0, y1);
+      } else {   // rows of odd length: every other row starts on an odd element
+        dst[i * 8] = __float2bfloat16_rn(y0);
+        dst[i * 8 + 1] = __float2bfloat16_rn(y1);
+      }
+    }
   }
 }
 
@@ -278,7 +250,7 @@ template <int NV>
 int launch_expanded(const void* qn, const float* qr, const void* kx, const void* vx, const void* kr_cache, int64_t S,
                     const int32_t* slot, const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count,
                     const int32_t* tile_kv_row, int n_tiles, int64_t n, int H, int dn, int dr, float scale, const void* sink,
-                    const float* gate, void* out, cudaStream_t st) {
+                    const float* gate, void* out, int64_t ldk, int64_t ldv, int window, int64_t ld_out, cudaStream_t st) {
   using T = __nv_bfloat16;
   const size_t smem = ((size_t)kPM * (dn + 2 * dr + kPad) + (size_t)kPN * (dn + dr + kPad) + (size_t)kPN * (16 * NV + kPad)) * 2;
   auto kern = latent_attn_expanded_kernel<NV>;
@@ -292,7 +264,8 @@ int launch_expanded(const void* qn, const float* qr, const void* kx, const void*
   dim3 grid((unsigned)n_tiles, (unsigned)H);
   kern<<<grid, kPWarps * 32, smem, st>>>(static_cast<const T*>(qn), qr, static_cast<const T*>(kx), static_cast<const T*>(vx),
                                          static_cast<const T*>(kr_cache), S, slot, pos, tile_first, tile_count, tile_kv_row, n, H,
-                                         dn, dr, scale, static_cast<const T*>(sink), gate, static_cast<T*>(out));
+                                         dn, dr, scale, static_cast<const T*>(sink), gate, static_cast<T*>(out), ldk, ldv, window,
+                                         ld_out);
   return lm_launch_status();
 }
 
@@ -304,6 +277,20 @@ extern "C" int ao_lm_latent_attention_expanded_plan(int dt, int dn, int dr, int 
   return AO_B200_OK;
 }
 
+static int dispatch_expanded(const void* qn, const float* qr, const void* kx, const void* vx, const void* kr, int64_t S,
+                             const int32_t* slot, const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count,
+                             const int32_t* tile_kv_row, int n_tiles, int64_t n, int H, int dn, int dr, int dv, float scale,
+                             const void* sink, const float* gate, void* out, int64_t ldk, int64_t ldv, int window, int64_t ld_out,
+                             cudaStream_t st) {
+#define LM_XP(NV)                                                                                                                  \
+  case NV:                                                                                                                         \
+    return launch_expanded<NV>(qn, qr, kx, vx, kr, S, slot, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, scale, \
+                               sink, gate, out, ldk, ldv, window, ld_out, st);
+  switch (dv / 16) { LM_XP(1) LM_XP(2) LM_XP(3) LM_XP(4) LM_XP(5) LM_XP(6) LM_XP(7) LM_XP(8) }
+#undef LM_XP
+  return AO_B200_ERR_UNSUPPORTED;
+}
+
 extern "C" int ao_lm_latent_attention_expanded(const void* qn, const float* qr, const void* kx, const void* vx,
                                                const void* kr_cache, int dt, int64_t S, const int32_t* slot,
                                                const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count,
@@ -313,12 +300,23 @@ extern "C" int ao_lm_latent_attention_expanded(const void* qn, const float* qr, 
   LM_CHECK_ARG((qr && kr_cache) || dr == 0);
   LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && H <= 65535 && S > 0);
   if (!expanded_ok(dt, dn, dr, dv)) return AO_B200_ERR_UNSUPPORTED;
-  const cudaStream_t st = lm_stream(stream);
-#define LM_XP(NV)                                                                                                          \
-  case NV:                                                                                                                 \
-    return launch_expanded<NV>(qn, qr, kx, vx, kr_cache, S, slot, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, \
-                               dr, scale, sink, gate, out, st);
-  switch (dv / 16) { LM_XP(1) LM_XP(2) LM_XP(3) LM_XP(4) LM_XP(5) LM_XP(6) LM_XP(7) LM_XP(8) }
-#undef LM_XP
-  return AO_B200_ERR_UNSUPPORTED;
+  return dispatch_expanded(qn, qr, kx, vx, kr_cache, S, slot, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, dv, scale,
+                           sink, gate, out, (int64_t)H * dn, (int64_t)H * dv, 0x7fffffff, (int64_t)H * dv, lm_stream(stream));
+}
+
+extern "C" int ao_lm_window_latent_attention_expanded(const void* qn, const float* qr, const void* kx, int64_t ldk, const void* vx,
+                                                      int64_t ldv, const void* kr, int dt, const int32_t* pos,
+                                                      const int32_t* tile_first, const int32_t* tile_count,
+                                                      const int32_t* tile_kv_row, int n_tiles, int64_t n, int H, int dn, int dr,
+                                                      int dv, float scale, int window, const void* sink, const float* gate,
+                                                      void* out, int64_t ld_out, void* stream) {
+  LM_CHECK_ARG(qn && kx && vx && pos && tile_first && tile_count && tile_kv_row && out && ((qr && kr) || dr == 0));
+  LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && H <= 65535 && window > 0 && ldk >= (int64_t)H * dn && ldv >= (int64_t)H * dv && ld_out >= (int64_t)H * dv);
+  if (!expanded_ok(dt, dn, dr, dv)) return AO_B200_ERR_UNSUPPORTED;
+  // 16-byte copies of queries, keys and values; the result is stored in pairs when its rows allow it
+  LM_CHECK_ARG(ldk % 8 == 0 && ldv % 8 == 0 && reinterpret_cast<uintptr_t>(qn) % 16 == 0 && reinterpret_cast<uintptr_t>(qr) % 16 == 0 &&
+               reinterpret_cast<uintptr_t>(kx) % 16 == 0 && reinterpret_cast<uintptr_t>(vx) % 16 == 0 &&
+               reinterpret_cast<uintptr_t>(kr) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 4 == 0);
+  return dispatch_expanded(qn, qr, kx, vx, kr, 0, nullptr, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, dv, scale,
+                           sink, gate, out, ldk, ldv, window, ld_out, lm_stream(stream));
 }

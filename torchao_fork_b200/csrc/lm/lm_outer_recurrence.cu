@@ -400,8 +400,8 @@ __global__ void conv_state_save_kernel(const float* __restrict__ x, int64_t ldx,
 // with the norm taken over each of `groups` equal parts of the row.  grid (rows, groups).
 template <typename T>
 __global__ void gated_group_norm_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ gate, int64_t ldg,
-                                        int mode, int64_t width, int groups, const T* __restrict__ weight, float eps,
-                                        T* __restrict__ out) {
+                                        int mode, int64_t width, int groups, const T* __restrict__ weight, int shared_weight,
+                                        float eps, T* __restrict__ out, int64_t ld_out) {
   __shared__ float scratch[33];
   const int64_t t = blockIdx.x, per = width / groups, c0 = (int64_t)blockIdx.y * per;
   const float* yr = y + t * ldy + c0;
@@ -420,14 +420,14 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, int64_t ldy
   for (int64_t c = threadIdx.x; c < per; c += blockDim.x) {
     const float z = gr[c];
     float v = yr[c];
-    const float wt = weight ? ldf(weight + c0 + c) : 1.f;
+    const float wt = weight ? ldf(weight + (shared_weight ? 0 : c0) + c) : 1.f;
     if (mode == 1)
       v = v * (z / (1.f + expf(-z))) * k * wt;
     else if (mode == 2)
       v = v * k * wt * (z / (1.f + expf(-z)));
     else
       v = v * k * wt / (1.f + expf(-z));
-    stf(out + t * width + c0 + c, v);
+    stf(out + t * ld_out + c0 + c, v);
   }
 }
 
@@ -437,8 +437,8 @@ constexpr int kGroupPerLane = 16;     // groups of up to 32 * 16 values
 template <typename T>
 __global__ void __launch_bounds__(256) gated_group_norm_warp_kernel(const float* __restrict__ y, int64_t ldy,
                                                                    const float* __restrict__ gate, int64_t ldg, int mode,
-                                                                   int64_t width, int groups, const T* __restrict__ weight, float eps,
-                                                                   T* __restrict__ out) {
+                                                                   int64_t width, int groups, const T* __restrict__ weight,
+                                                                   int shared_weight, float eps, T* __restrict__ out, int64_t ld_out) {
   const int lane = threadIdx.x & 31, grp = blockIdx.y * 8 + (threadIdx.x >> 5);
   if (grp >= groups) return;
   const int64_t t = blockIdx.x;
@@ -460,13 +460,13 @@ __global__ void __launch_bounds__(256) gated_group_norm_warp_kernel(const float*
   for (int e = 0; e < kGroupPerLane; ++e) {
     const int c = lane + 32 * e;
     if (c >= per) continue;
-    const float wt = weight ? ldf(weight + c0 + c) : 1.f;
+    const float wt = weight ? ldf(weight + (shared_weight ? 0 : c0) + c) : 1.f;
     float r = v[e] * k * wt;
     if (mode == 2)
       r *= z[e] / (1.f + expf(-z[e]));
     else if (mode == 0)
       r /= 1.f + expf(-z[e]);
-    stf(out + t * width + c0 + c, r);
+    stf(out + t * ld_out + c0 + c, r);
   }
 }
 
@@ -523,16 +523,24 @@ extern "C" int ao_lm_conv_state_save(const float* x, int64_t ldx, int64_t n, int
   return lm_launch_status();
 }
 
-extern "C" int ao_lm_gated_group_norm(const float* y, int64_t ldy, const float* gate, int64_t ldg, int mode, int64_t n,
-                                      int64_t width, int groups, const void* weight, int dt, float eps, void* out, void* stream) {
-  LM_CHECK_ARG(y && gate && out && n > 0 && width > 0 && groups > 0 && groups <= 65535 && width % groups == 0);
+extern "C" int ao_lm_gated_group_norm_rows(const float* y, int64_t ldy, const float* gate, int64_t ldg, int mode, int64_t n,
+                                           int64_t width, int groups, const void* weight, int shared_weight, int dt, float eps,
+                                           void* out, int64_t ld_out, void* stream) {
+  LM_CHECK_ARG(y && gate && out && n > 0 && width > 0 && groups > 0 && groups <= 65535 && width % groups == 0 && ld_out >= width);
   LM_CHECK_ARG(mode == 0 || mode == 1 || mode == 2);
   if (groups > 1 && width / groups <= 32 * kGroupPerLane) {
     LM_DISPATCH(dt, gated_group_norm_warp_kernel<T><<<dim3((unsigned)n, (unsigned)((groups + 7) / 8)), 256, 0, lm_stream(stream)>>>(
-                        y, ldy, gate, ldg, mode, width, groups, static_cast<const T*>(weight), eps, static_cast<T*>(out)));
+                        y, ldy, gate, ldg, mode, width, groups, static_cast<const T*>(weight), shared_weight, eps,
+                        static_cast<T*>(out), ld_out));
     return lm_launch_status();
   }
   LM_DISPATCH(dt, gated_group_norm_kernel<T><<<dim3((unsigned)n, (unsigned)groups), 256, 0, lm_stream(stream)>>>(
-                      y, ldy, gate, ldg, mode, width, groups, static_cast<const T*>(weight), eps, static_cast<T*>(out)));
+                      y, ldy, gate, ldg, mode, width, groups, static_cast<const T*>(weight), shared_weight, eps, static_cast<T*>(out),
+                      ld_out));
   return lm_launch_status();
+}
+
+extern "C" int ao_lm_gated_group_norm(const float* y, int64_t ldy, const float* gate, int64_t ldg, int mode, int64_t n,
+                                      int64_t width, int groups, const void* weight, int dt, float eps, void* out, void* stream) {
+  return ao_lm_gated_group_norm_rows(y, ldy, gate, ldg, mode, n, width, groups, weight, 0, dt, eps, out, width, stream);
 }

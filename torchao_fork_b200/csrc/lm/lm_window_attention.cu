@@ -23,13 +23,15 @@ constexpr int kMaxDvLane = 8;    // value size <= 32 * kMaxDvLane
 constexpr int kPairs = kWarps * kSlots;
 
 // Projection row -> biased, rotated queries (fp32 [n][q_heads][d]) and keys (storage type [n][k_heads][d]), biased values
-// (storage type [n][v_width]).  k_heads == 0: a layer that borrows its keys and values projects queries only.
+// (storage type [n][v_width]).  k_heads == 0: a layer that borrows its keys and values projects queries only.  amp multiplies
+// cosine and sine; v_first: another layer's values of the same rows, mixed in with weight v_mix.
 template <typename T>
 __global__ void qkv_rotary_prep_kernel(const float* __restrict__ proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off,
                                        const T* __restrict__ q_bias, const T* __restrict__ k_bias, const T* __restrict__ v_bias,
                                        const int32_t* __restrict__ pos, const float* __restrict__ inv_freq, int rot_dims,
-                                       int pairing, int q_heads, int k_heads, int d, int v_width, float* __restrict__ qn,
-                                       T* __restrict__ kn, T* __restrict__ vn) {
+                                       int pairing, float amp, const T* __restrict__ v_first, float v_mix, int q_heads,
+                                       int k_heads, int d, int v_width, float* __restrict__ qn, T* __restrict__ kn,
+                                       T* __restrict__ vn) {
   const int64_t t = blockIdx.x;
   const float p = (float)pos[t];
   const float* row = proj + t * ld;
@@ -48,6 +50,7 @@ __global__ void qkv_rotary_prep_kernel(const float* __restrict__ proj, int64_t l
       const float u = src[ia] + (bias ? ldf(bias + ho + ia) : 0.f), v = src[ib] + (bias ? ldf(bias + ho + ib) : 0.f);
       float sn, cs;
       sincosf(p * inv_freq[e], &sn, &cs);
+      sn *= amp, cs *= amp;
       va = u * cs - v * sn, vb = v * cs + u * sn;
     } else {
       ia = rot_dims + (e - half);
@@ -64,8 +67,11 @@ __global__ void qkv_rotary_prep_kernel(const float* __restrict__ proj, int64_t l
     }
   }
   if (k_heads > 0)
-    for (int c = tid; c < v_width; c += nth)
-      stf(vn + t * v_width + c, row[v_off + c] + (v_bias ? ldf(v_bias + c) : 0.f));
+    for (int c = tid; c < v_width; c += nth) {
+      float v = row[v_off + c] + (v_bias ? ldf(v_bias + c) : 0.f);
+      if (v_first) v = fmaf(v_mix, ldf(v_first + t * v_width + c), (1.f - v_mix) * v);
+      stf(vn + t * v_width + c, v);
+    }
 }
 
 template <typename T>
@@ -431,10 +437,11 @@ int launch_window(const WinArgs& a, int n_tiles, size_t smem, cudaStream_t st) {
 
 }  // namespace
 
-extern "C" int ao_lm_qkv_rotary_prep(const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, const void* q_bias,
-                                     const void* k_bias, const void* v_bias, const int32_t* pos, const float* inv_freq,
-                                     int rot_dims, int pairing, int64_t n, int q_heads, int k_heads, int d, int v_width, int dt,
-                                     float* qn, void* kn, void* vn, void* stream) {
+extern "C" int ao_lm_qkv_rotary_mix_prep(const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off,
+                                         const void* q_bias, const void* k_bias, const void* v_bias, const int32_t* pos,
+                                         const float* inv_freq, int rot_dims, int pairing, float amp, const void* v_first, float v_mix,
+                                         int64_t n, int q_heads, int k_heads, int d, int v_width, int dt, float* qn, void* kn, void* vn,
+                                         void* stream) {
   LM_CHECK_ARG(proj && pos && qn && n > 0 && q_heads > 0 && k_heads >= 0 && d > 0 && (k_heads == 0 || (kn && vn && v_width > 0)));
   LM_CHECK_ARG(rot_dims >= 0 && rot_dims <= d && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq) && (pairing == 0 || pairing == 1));
   // few rows (decoded tokens): several CTAs per row, so that no thread walks more than a few coordinates
@@ -443,9 +450,17 @@ extern "C" int ao_lm_qkv_rotary_prep(const float* proj, int64_t ld, int64_t q_of
   const unsigned parts = n < 296 ? (unsigned)(want > room ? room : want < 1 ? 1 : want) : 1u;
   LM_DISPATCH(dt, qkv_rotary_prep_kernel<T><<<dim3((unsigned)n, parts), 256, 0, lm_stream(stream)>>>(
                       proj, ld, q_off, k_off, v_off, static_cast<const T*>(q_bias), static_cast<const T*>(k_bias),
-                      static_cast<const T*>(v_bias), pos, inv_freq, rot_dims, pairing, q_heads, k_heads, d, v_width, qn,
-                      static_cast<T*>(kn), static_cast<T*>(vn)));
+                      static_cast<const T*>(v_bias), pos, inv_freq, rot_dims, pairing, amp, static_cast<const T*>(v_first), v_mix,
+                      q_heads, k_heads, d, v_width, qn, static_cast<T*>(kn), static_cast<T*>(vn)));
   return lm_launch_status();
+}
+
+extern "C" int ao_lm_qkv_rotary_prep(const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, const void* q_bias,
+                                     const void* k_bias, const void* v_bias, const int32_t* pos, const float* inv_freq,
+                                     int rot_dims, int pairing, int64_t n, int q_heads, int k_heads, int d, int v_width, int dt,
+                                     float* qn, void* kn, void* vn, void* stream) {
+  return ao_lm_qkv_rotary_mix_prep(proj, ld, q_off, k_off, v_off, q_bias, k_bias, v_bias, pos, inv_freq, rot_dims, pairing, 1.f,
+                                   nullptr, 0.f, n, q_heads, k_heads, d, v_width, dt, qn, kn, vn, stream);
 }
 
 extern "C" int ao_lm_window_append(const void* kn, const void* vn, int64_t n, int64_t k_row, int64_t v_row, int ring,
