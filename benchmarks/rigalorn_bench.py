@@ -213,7 +213,7 @@ class Bench:
         prep(n, self.pos)
         seg, cnt = self.zero, self.i32([n])
         flops = 6.0 * n * H * d * dv       # two products with the state and the update
-        for key, rows, count, pos, block in (("delta_prefill", n, cnt, self.pos, 4), ("delta_prefill_one_at_a_time", n, cnt, self.pos, 1),
+        for key, rows, count, pos, block in (("delta_prefill", n, cnt, self.pos, 8), ("delta_prefill_one_at_a_time", n, cnt, self.pos, 1),
                                              ("delta_decode", 1, self.one, self.last, 1)):
             ms = self.call("delta_recurrence", qk, v, gb, H, G, dp, dv, state, self.slot, pos, seg, count, 1, block, proj, ld, C, taps, mem, out)
             if rows > 1:

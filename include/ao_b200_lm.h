@@ -468,8 +468,8 @@ AO_B200_API int ao_lm_delta_prep(const float* proj, int64_t ld, int64_t conv_off
 
 /* Gated delta rule per head (fp32 state[slots][H][dv][dp], zeros at position 0): S <- g S; u = beta (v - S^T k);
  * S <- S + k u^T; out[t][h] = S^T q (fp32 [n][H dv]); head h reads group h / (H / G) of q and k.  seg_first / seg_count: the
- * step's segments, whole.  block: tokens folded in at a time, 4 (segments of several rows) or 1; the same sums in another
- * order.  With conv_x (fp32, row stride ld_conv), the last taps - 1 rows of every segment of its `channels` values become
+ * step's segments, whole.  block: tokens folded in at a time, 8 (segments of several rows; 4 where dp > 256) or 1; the same
+ * sums in another order.  dp <= 1024.  With conv_x (fp32, row stride ld_conv), the last taps - 1 rows of every segment of its `channels` values become
  * conv_state[slot] (the memory of the convolution that made q, k and v). */
 AO_B200_API int ao_lm_delta_recurrence(const float* qk, const float* v, const float* gb, int H, int G, int dp, int dv, float* state,
                                        const int32_t* slot, const int32_t* pos, const int32_t* seg_first, const int32_t* seg_count,

@@ -201,7 +201,7 @@ def _delta_run(proj, conv_w, a_log, dt_bias, m, cuts, block=None, slots=3, slot=
                                         dt, 1e-6, d ** -0.5, _p(qk), _p(v), _p(gb), _st()), "prep")
         out = torch.zeros(c, H * dv, device="cuda")
         lib.lm_check(L.ao_lm_delta_recurrence(_p(qk), _p(v), _p(gb), H, G, dp, dv, _p(state), _p(sd), _p(pd), _p(sf), _p(sc), 1,
-                                              block or (1 if c == 1 else 4), _p(x), ld, C, taps, _p(mem), _p(out), _st()), "recurrence")
+                                              block or (1 if c == 1 else 8), _p(x), ld, C, taps, _p(mem), _p(out), _st()), "recurrence")
         parts.append((qk[..., :d], v.view(c, H, dv), gb, out.view(c, H, dv)))
     assert float(state[:slot].min()) == 7.0 and float(mem[:slot].min()) == 5.0      # other slots untouched
     return [torch.cat([p[i] for p in parts]) for i in range(4)]
@@ -223,12 +223,12 @@ def _delta_case(H, G, d, dv, taps, T=75):
     return m, proj, conv, a_log, dt_bias, ref, O.delta_recurrence(*ref)
 
 
-@pytest.mark.parametrize("H,G,d,dv,taps", [(2, 1, 8, 8, 4), (3, 3, 5, 7, 2), (1, 1, 64, 40, 1), (4, 2, 30, 33, 3), (2, 2, 128, 16, 4), (6, 2, 100, 64, 5),
+@pytest.mark.parametrize("H,G,d,dv,taps", [(2, 1, 8, 8, 4), (3, 3, 5, 7, 2), (1, 1, 12, 8, 2), (2, 2, 160, 12, 3), (3, 1, 132, 20, 2), (1, 1, 64, 40, 1), (4, 2, 30, 33, 3), (2, 2, 128, 16, 4), (6, 2, 100, 64, 5),
                                            (1, 1, 200, 9, 4), (1, 1, 300, 5, 4), (1, 1, 600, 3, 2), (2, 1, 1, 1, 7)])
 def test_delta_rule_with_its_convolutions_in_portions(H, G, d, dv, taps):
     T = 75
     m, proj, conv, a_log, dt_bias, (q, k, v, g, beta), ref = _delta_case(H, G, d, dv, taps, T)
-    for cuts, block in ([(0, T)], None), (_cuts(T, [1]), None), (_cuts(T, [1]), 4), (_cuts(T, [2, 17, 1, 33]), None), (_cuts(T, [2]), None), ([(0, T)], 1):
+    for cuts, block in ([(0, T)], None), (_cuts(T, [1]), None), (_cuts(T, [1]), 8), (_cuts(T, [2, 17, 1, 33]), None), (_cuts(T, [2]), None), ([(0, T)], 1):
         qk, vv, gb, out = _delta_run(proj, conv, a_log, dt_bias, m, cuts, block)
         assert _close(qk[:, 0], q, 1e-5) and _close(qk[:, 1], k, 1e-5) and _close(vv, v, 1e-5), (cuts[:3], block)
         assert _close(gb[..., 0], g, 1e-5) and _close(gb[..., 1], beta, 1e-5)
@@ -251,7 +251,7 @@ def test_delta_rule_several_segments_of_unequal_length_in_one_launch():
         r = torch.tensor(rows, device="cuda")
         a, b, c = qk[r].contiguous(), vd[r].contiguous(), gb[r].contiguous()
         out = torch.zeros(len(rows), H * dv, device="cuda")
-        lib.lm_check(L.ao_lm_delta_recurrence(_p(a), _p(b), _p(c), H, G, d, dv, _p(state), _p(sd), _p(pd), _p(sf), _p(sc), len(segs), 4, None, 0, 0,
+        lib.lm_check(L.ao_lm_delta_recurrence(_p(a), _p(b), _p(c), H, G, d, dv, _p(state), _p(sd), _p(pd), _p(sf), _p(sc), len(segs), 8, None, 0, 0,
                                               1, None, _p(out), _st()), "recurrence")
         at = 0
         for s, p0, n in segs:
@@ -282,7 +282,7 @@ def test_delta_rule_remembers_for_hundreds_of_tokens_and_overwrites_one_key():
                 qk = torch.stack([q[a:a + c], keys[a:a + c]], 1).cuda()
                 vd, gb, out = v[a:a + c].cuda(), torch.ones(c, 1, 2, device="cuda"), torch.zeros(c, dv, device="cuda")
                 lib.lm_check(L.ao_lm_delta_recurrence(_p(qk), _p(vd), _p(gb), 1, 1, d, dv, _p(state), _p(sd), _p(pd), _p(sf), _p(sc), 1,
-                                                      1 if c == 1 else 4, None, 0, 0, 1, None, _p(out), _st()), "recurrence")
+                                                      1 if c == 1 else 8, None, 0, 0, 1, None, _p(out), _st()), "recurrence")
                 outs.append(out)
             assert _close(torch.cat(outs)[-1], want, 1e-4), cuts[:2]
 

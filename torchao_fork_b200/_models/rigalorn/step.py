@@ -189,7 +189,7 @@ class StepEngine(SegmentStepEngine):
         rec = torch.empty(n, H * dv, **f32)
         sf, sc, ns = meta.seg
         _lib.lm_check(L.ao_lm_delta_recurrence(_p(qk), _p(v), _p(gb), H, G, dp, dv, _p(ls.mat.s), _p(meta.slot), _p(meta.pos), _p(sf), _p(sc),
-                                               ns, 1 if ns == n else 4, _p(proj), lay.ld, a.channels, a.taps, _p(ls.conv.x), _p(rec), st),
+                                               ns, 1 if ns == n else 8, _p(proj), lay.ld, a.channels, a.taps, _p(ls.conv.x), _p(rec), st),
                       "delta_recurrence")
         _lib.lm_check(L.ao_lm_gated_group_norm_rows(_p(rec), H * dv, proj.data_ptr() + 4 * lay.g_off, lay.ld, GATE_SILU_AFTER_NORM, n, H * dv,
                                                     H, _p(lay.mix_norm), 1, dt, self.cfg.norm_eps, _p(row), row.shape[1], st),
