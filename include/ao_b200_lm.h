@@ -509,6 +509,56 @@ AO_B200_API int ao_lm_window_latent_attention_expanded(const void* qn, const flo
 AO_B200_API int ao_lm_latent_rows_gather(const int32_t* src, int64_t rows, const void* c, const void* kr, const void* ring_c,
                                          const void* ring_kr, int dt, int R, int dr, void* out_c, void* out_kr, void* stream);
 
+/* ---------------------------------------------------------------------------------------------------------------
+ * Layer norms on both sides of every sublayer, spans of layers run several times with the embedding output fed in again, a
+ * hashed embedding of token pairs, normed and rotated queries and keys, latent attention with an element-wise gate.
+ */
+
+/* v = y[t] + y_bias (fp32 [n] rows of stride ld_y, fp32 [width]; bias null: none);  with post_w (`dt`), v = LN(v) * post_w, LN(u) =
+ * (u - mean) / sqrt(mean squared deviation + eps);  x[t] = (replace ? 0 : x[t]) + v + add_rows[t] (fp32, stride ld_add; null:
+ * none);  out[t] (`dt`, stride ld_out; null: none) = next_w ? LN(x[t]) * next_w : x[t].  y null: x is only read. */
+AO_B200_API int ao_lm_post_layer_norm_residual(float* x, const float* y, int64_t ld_y, const float* y_bias, const void* post_w,
+                                               const float* add_rows, int64_t ld_add, int replace, const void* next_w, int dt, float eps,
+                                               int64_t n, int64_t width, void* out, int64_t ld_out, void* stream);
+
+/* x[t] = table[tok[t]] * scale + bigram[r] (fp32; out, when not null, the same in `dt`), r = (previous * mul_prev + tok[t] * mul_cur)
+ * mod buckets, for the first token of a sequence r = buckets (the table's last row); bigram null: no second term.  The previous
+ * token of a segment's first row is last[slot]; the segment's last token replaces it. */
+AO_B200_API int ao_lm_embed_bigram(const void* table, const void* bigram, int dt, const int64_t* tok, int64_t n, int64_t width,
+                                   float scale, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int64_t* last, const int32_t* slot,
+                                   const int32_t* pos, const int32_t* back, const int32_t* ahead, float* x, void* out, void* stream);
+
+/* ao_lm_qkv_rotary_prep with every query and key head divided by its root mean square (eps inside the root) and multiplied by
+ * q_weight / k_weight (`dt` [d]; null: no norm) between bias and rotation, and amp on cosine and sine.  With ring_k / ring_v the
+ * keys and values also go to row pos % ring of the slot: only for steps that bring ONE row per sequence (a longer segment's
+ * first rows may still need the ring rows that its last rows replace; use ao_lm_window_append there). */
+AO_B200_API int ao_lm_qkv_norm_rotary_prep(const float* proj, int64_t ld, int64_t q_off, int64_t k_off, int64_t v_off, const void* q_bias,
+                                           const void* k_bias, const void* v_bias, const void* q_weight, const void* k_weight, float eps,
+                                           const int32_t* pos, const float* inv_freq, int rot_dims, int pairing, float amp, int64_t n, int H,
+                                           int G, int d, int v_width, int dt, float* qn, void* kn, void* vn, const int32_t* slot, int ring,
+                                           void* ring_k, void* ring_v, void* stream);
+
+/* ao_lm_latent_low_prep that also writes c and kr to row pos[t] of the slot's cache [slots][S][R] / [slots][S][dr] (c_cache null:
+ * does not); a cache that never wraps needs no append launch then. */
+AO_B200_API int ao_lm_latent_low_prep_store(const float* proj, int64_t ld, int64_t n, int64_t q_off, int Rq, int64_t kv_off, int R, int dr,
+                                            const void* q_norm, const void* c_norm, int dt, float eps, int rot_dims, const float* inv_freq,
+                                            float amp, const int32_t* pos, const int32_t* slot, int64_t S, void* cq, void* c, void* kr,
+                                            void* c_cache, void* kr_cache, void* stream);
+
+/* ao_lm_window_latent_attention_expanded whose result is multiplied by sigmoid(gate_rows[t][h * dv + c]) (fp32 logits, row stride
+ * ld_gate; null: no gate). */
+AO_B200_API int ao_lm_gated_latent_attention_expanded(const void* qn, const float* qr, const void* kx, int64_t ldk, const void* vx,
+                                                      int64_t ldv, const void* kr, int dt, const int32_t* pos, const int32_t* tile_first,
+                                                      const int32_t* tile_count, const int32_t* tile_kv_row, int n_tiles, int64_t n, int H,
+                                                      int dn, int dr, int dv, float scale, int window, const void* sink,
+                                                      const float* gate_rows, int64_t ld_gate, void* out, int64_t ld_out, void* stream);
+/* The folded form's way back, for few rows: out[t][h * dv + j] = sigmoid(gate[t][h * dv + j]) * sum_r uv[h][j][r] * olat[t][h][r]
+ * (olat, uv, out in `dt`; gate fp32 logits with row stride ld_gate, null: none).  ao_lm_sigmoid_gate_rows: y *= sigmoid(gate). */
+AO_B200_API int ao_lm_latent_value_up(const void* olat, const void* uv, int dt, int64_t n, int H, int R, int dv, const float* gate,
+                                      int64_t ld_gate, void* out, int64_t ld_out, void* stream);
+AO_B200_API int ao_lm_sigmoid_gate_rows(const float* gate, int64_t ld_gate, int64_t n, int64_t cols, void* y, int64_t ld, int dt,
+                                        void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -524,7 +524,7 @@ def test_either_attention_form_for_every_portion_and_batch(monkeypatch, min_rows
 
 
 def test_pieces_cut_inside_a_step_and_the_folded_form_when_expanded_rows_would_be_too_many(monkeypatch):
-    import torchao_fork_b200._models.rigalorn.step as RS
+    import torchao_fork_b200._models.softmax_step as RS
     import torchao_fork_b200._models.segment_step as S
     for make in (_mixed, _tensor):
         cfg = make()

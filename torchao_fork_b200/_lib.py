@@ -226,6 +226,16 @@ LM_SIGNATURES = {
     "ao_lm_window_latent_attention_expanded": [_vp, _vp, _vp, _i64, _vp, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i64, _i32, _i32,
                                                _i32, _i32, _f32, _i32, _vp, _vp, _vp, _i64, _vp],
     "ao_lm_latent_rows_gather": [_vp, _i64, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _vp, _vp, _vp],
+    "ao_lm_post_layer_norm_residual": [_vp, _vp, _i64, _vp, _vp, _vp, _i64, _i32, _vp, _i32, _f32, _i64, _i64, _vp, _i64, _vp],
+    "ao_lm_embed_bigram": [_vp, _vp, _i32, _vp, _i64, _i64, _f32, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
+    "ao_lm_qkv_norm_rotary_prep": [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _vp, _f32, _vp, _vp, _i32, _i32, _f32, _i64, _i32, _i32,
+                                   _i32, _i32, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp],
+    "ao_lm_latent_low_prep_store": [_vp, _i64, _i64, _i64, _i32, _i64, _i32, _i32, _vp, _vp, _i32, _f32, _i32, _vp, _f32, _vp, _vp, _i64,
+                                    _vp, _vp, _vp, _vp, _vp, _vp],
+    "ao_lm_gated_latent_attention_expanded": [_vp, _vp, _vp, _i64, _vp, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i64, _i32, _i32, _i32,
+                                              _i32, _f32, _i32, _vp, _vp, _i64, _vp, _i64, _vp],
+    "ao_lm_latent_value_up": [_vp, _vp, _i32, _i64, _i32, _i32, _i32, _vp, _i64, _vp, _i64, _vp],
+    "ao_lm_sigmoid_gate_rows": [_vp, _i64, _i64, _i64, _vp, _i64, _i32, _vp],
 }
 _LM_RESTYPES = {"ao_lm_last_cuda_error": ctypes.c_char_p, "ao_lm_latent_attention_workspace_bytes": _i64, "ao_lm_scan_workspace_bytes": _i64, "ao_lm_outer_recurrence_workspace_bytes": _i64, "ao_lm_channel_recurrence_workspace_bytes": _i64, "ao_lm_window_attention_workspace_bytes": _i64,
                 "ao_lm_chunk_attention_workspace_bytes": _i64}

@@ -123,6 +123,18 @@ class TokenShiftState(nn.Module):
         self.prev = new
 
 
+class LastTokenState(nn.Module):
+    """The id of a sequence's last token, per slot: an embedding that hashes token pairs reads it for the next step's first
+    token.  A sequence's first token does not read it, so a reused slot needs no clearing."""
+
+    def __init__(self, n_slots, device=None):
+        super().__init__()
+        self.register_buffer("token", torch.zeros(n_slots, dtype=torch.int64, device=device))
+
+    def grow(self, n_slots):
+        self.token = _grown(self.token, n_slots)
+
+
 def _grown(old: torch.Tensor, n_slots: int) -> torch.Tensor:
     new = torch.zeros(n_slots, *old.shape[1:], dtype=old.dtype, device=old.device)
     new[: old.shape[0]] = old

@@ -51,6 +51,9 @@ def _load_builtin():
     from .rigalorn import model as _rigalorn
     register(Family("rigalorn", from_folder=_rigalorn.Rigalorn.from_checkpoint, from_name=_rigalorn.Rigalorn.from_name,
                     names=lambda: list(_rigalorn.rigalorn_configs)))
+    from .sozanex import model as _sozanex
+    register(Family("sozanex", from_folder=_sozanex.Sozanex.from_checkpoint, from_name=_sozanex.Sozanex.from_name,
+                    names=lambda: list(_sozanex.sozanex_configs)))
 
 
 def architecture_of(folder) -> str:

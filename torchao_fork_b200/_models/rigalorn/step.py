@@ -26,81 +26,17 @@ storage types.
 `StepEngine.step` is what prefill, the trace runner and tests call; `GraphDecodeEngine` wraps the same layer loop for
 one token per sequence with all metadata in device memory, captured into a CUDA graph.
 """
-import ctypes
-
-import numpy as np
 import torch
 
 from ... import _lib
-from ..segment_step import GraphDecodeEngine, SegmentStepEngine, StepMeta, _p  # noqa: F401
+from ..segment_step import GraphDecodeEngine, StepMeta, _p  # noqa: F401
+from ..softmax_step import PAIR_HALVES, SoftmaxStepEngine
 from .model import UNIT_EPS, Rigalorn
 
-PAIR_HALVES = 1                           # rotation couples (i, i + dims / 2)
 GATE_SILU_AFTER_NORM = 2                  # mode of gated_group_norm
-# prompt portions attend over expanded keys and values of at most this many bytes per layer; beyond it in the folded form
-EXPAND_MAX_BYTES = 4 << 30
 
 
-class StepEngine(SegmentStepEngine):
-    def __init__(self, model: Rigalorn):
-        super().__init__(model)
-        self.windows = sorted({s[-1] for s in self.attn_keys if s[0] == "latent"})
-
-    # ------------------------------------------------------------------------------------------------ plans
-    def _shape(self, la, ls):
-        a = la.mixer
-        if la.type == "attention":
-            return ("window", a.heads, a.kv_heads, a.dim, a.vdim)
-        return ("latent", a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, min(a.window, ls.latent.c.shape[1]))
-
-    def _attention_shapes(self):
-        return sorted({self._shape(la, ls) for la, ls in zip(self.cfg.layers, self.m.run_state) if la.type != "delta"})
-
-    def _attention_plan(self, shape):
-        rows, prompt = ctypes.c_int(), ctypes.c_int()
-        if shape[0] == "window":
-            _, H, G, d, dv = shape
-            _lib.lm_check(self.L.ao_lm_window_attention_plan(self.dt, 1, H, G, d, dv, ctypes.byref(rows)), "window_attention_plan")
-            _lib.lm_check(self.L.ao_lm_window_attention_prompt_plan(self.dt, 1, H, G, d, dv, ctypes.byref(prompt)), "window_attention_prompt_plan")
-        else:
-            _, H, dn, dr, dv, R, _ = shape
-            _lib.lm_check(self.L.ao_lm_latent_attention_plan(self.dt, H, R, dr, ctypes.byref(rows)), "latent_attention_plan")
-            _lib.lm_check(self.L.ao_lm_latent_attention_expanded_plan(self.dt, dn, dr, dv, ctypes.byref(prompt)), "latent_attention_expanded_plan")
-        return rows.value, 1 << 30, prompt.value      # tiles may cross any position
-
-    @staticmethod
-    def _history(pos0, window):
-        """Keys from earlier steps that a segment starting at position pos0 can see."""
-        return np.minimum(pos0, window - 1)
-
-    def _prompt_form(self, shape, starts, counts, pos):
-        if shape[0] != "latent":
-            return True
-        _, H, dn, _, dv, _, window = shape
-        return int((self._history(pos[starts], window) + counts).sum()) * H * (dn + dv) * 2 <= EXPAND_MAX_BYTES
-
-    def _piece_tables(self, starts, counts, slot, pos, forms, tiles):
-        """For every window of latent-attention layers that attend in the expanded form: ("rows", window) = where each
-        contiguous latent row comes from (absent when the step's own rows are all of them), ("key0", window) = per tile, the
-        row that key 0 of its sequence would have."""
-        out = {}
-        for shape, form in forms.items():
-            if shape[0] != "latent" or not form[2] or ("key0", shape[-1]) in out:
-                continue
-            window = shape[-1]
-            hist = self._history(pos[starts], window)
-            base = np.concatenate([[0], np.cumsum(hist + counts)[:-1]])            # a segment's first contiguous row
-            first = tiles[form][0]
-            seg = np.searchsorted(starts, first, side="right") - 1
-            out[("key0", window)] = (base - (pos[starts] - hist))[seg].astype(np.int32)
-            if hist.any():
-                parts = []
-                for s, c, h in zip(starts, counts, hist):
-                    p0 = int(pos[s])
-                    parts += [-1 - (int(slot[s]) * window + np.arange(p0 - h, p0) % window), np.arange(s, s + c)]
-                out[("rows", window)] = np.concatenate(parts).astype(np.int32)
-        return out
-
+class StepEngine(SoftmaxStepEngine):
     # ------------------------------------------------------------------------------------------------ layers
     def _norm(self, x, y, w, st):
         """x += y (None: nothing added); -> RMS norm of x with weight w in the model's dtype (w None: only the add)."""
@@ -161,20 +97,8 @@ class StepEngine(SegmentStepEngine):
         _lib.lm_check(L.ao_lm_qkv_rotary_mix_prep(_p(proj), lay.ld, lay.q_off, lay.k_off, lay.v_off, _p(lay.q_b), _p(lay.k_b), _p(lay.v_b),
                                                   _p(meta.pos), _p(lay.inv_freq), a.rot.dims, PAIR_HALVES, a.rot.amplitude, _p(v_first),
                                                   lay.lam, n, H, G, d, G * dv, dt, _p(qn), _p(kn), _p(vn), st), "qkv_rotary_mix_prep")
-        tf, tc, nt, tensor = meta.attn[self._shape(la, ls)]
-        window = min(a.window, cache.ring)
-        common = (_p(qn), _p(kn), _p(vn), _p(cache.k), _p(cache.v), _p(cache.k_first), _p(cache.v_first), cache.ring, 0, dt, _p(meta.slot),
-                  _p(meta.pos), _p(meta.back), _p(tf), _p(tc), nt, 1, H, G, d, dv, window, 0, a.scale, 0.0, 0, 0.0, 1.0)
-        c = 3
-        if tensor:      # prompt portions: the tensor-core form
-            _lib.lm_check(L.ao_lm_window_attention_prompt(*common, _p(row), row.shape[1], st), "window_attention_prompt")
-        else:
-            ns = self._splits(nt * G, window)    # few rows over a long window: the keys are shared out over more CTAs
-            ws = torch.empty(max(16, int(L.ao_lm_window_attention_workspace_bytes(nt, 1, H, G, dv, ns))), dtype=torch.uint8, device=dev)
-            _lib.lm_check(L.ao_lm_window_attention(*common, ns, _p(ws), ws.numel(), _p(row), row.shape[1], st), "window_attention")
-            c += 1 if ns > 1 else 0
-        _lib.lm_check(L.ao_lm_window_append(_p(kn), _p(vn), n, G * d, G * dv, cache.ring, 0, dt, _p(meta.slot), _p(meta.pos), _p(meta.ahead),
-                                            _p(cache.k), _p(cache.v), _p(cache.k_first), _p(cache.v_first), st), "window_append")
+        c = 2 + self._window_attend(a, self._shape(la, ls), cache, qn, kn, vn, row, meta, st)
+        self._window_append(a, cache, kn, vn, meta, st)
         return vn, c
 
     def _delta(self, lay, a, ls, proj, row, meta: StepMeta, st):
@@ -205,51 +129,11 @@ class StepEngine(SegmentStepEngine):
         rot = (a.rot.dims, _p(lay.inv_freq), a.rot.amplitude)
         _lib.lm_check(L.ao_lm_latent_low_prep(_p(proj), lay.ld, n, lay.q_off, Rq, lay.kv_off, R, dr, _p(lay.q_norm), _p(lay.c_norm), dt,
                                               self.cfg.norm_eps, *rot, _p(meta.pos), _p(cq), _p(c), _p(kr), st), "latent_low_prep")
-        q = self._mm_f32(cq, lay.uq)
-        qn, qr = torch.empty(H, n, dn, **act), torch.empty(n, H, dr, dtype=torch.float32, device=dev)
-        _lib.lm_check(L.ao_lm_latent_query_prep(_p(q), n, H, dn, dr, dt, *rot, _p(meta.pos), _p(qn), _p(qr), st), "latent_query_prep")
-        shape = self._shape(la, ls)
-        ring, window = cache.c.shape[1], shape[-1]
-        tf, tc, nt, tensor = meta.attn[shape]
-        launches = 4
-        if tensor:
-            launches += self._latent_expanded(lay, a, cache, c, kr, qn, qr, row, tf, tc, nt, window, meta, st)
-        else:
-            qa = self._bmm_f32(qn, lay.uk)                                             # fp32 [H][n][R]
-            ns = self._splits(nt * -(-H // 16), window)
-            ws = torch.empty(max(16, int(L.ao_lm_latent_attention_workspace_bytes(n, H, R, ns))), dtype=torch.uint8, device=dev)
-            olat = torch.empty(n, H, R, **act)
-            _lib.lm_check(L.ao_lm_window_latent_attention(_p(qa), _p(qr), _p(cache.c), _p(cache.kr), _p(c), _p(kr), dt, ring, _p(meta.slot),
-                                                          _p(meta.pos), _p(meta.back), _p(tf), _p(tc), nt, n, H, R, dr, a.scale, window,
-                                                          None, None, ns, _p(ws), ws.numel(), _p(olat), st), "window_latent_attention")
-            heads = row.as_strided((H, n, dv), (dv, row.shape[1], 1))
-            torch.bmm(olat.transpose(0, 1), lay.uv.transpose(1, 2), out=heads)
-            launches += 4 if ns > 1 else 3
-        _lib.lm_check(L.ao_lm_ring_append(_p(c), _p(kr), n, R, dr, ring, dt, _p(meta.slot), _p(meta.pos), _p(meta.ahead), _p(cache.c),
-                                          _p(cache.kr), st), "ring_append")
+        qn, qr = self._latent_queries(lay, a, cq, meta, st)
+        launches = 4 + self._latent_attend(lay, a, self._shape(la, ls), cache, c, kr, qn, qr, row, meta, st)
+        _lib.lm_check(L.ao_lm_ring_append(_p(c), _p(kr), n, R, dr, cache.c.shape[1], dt, _p(meta.slot), _p(meta.pos), _p(meta.ahead),
+                                          _p(cache.c), _p(cache.kr), st), "ring_append")
         return launches
-
-    def _latent_expanded(self, lay, a, cache, c, kr, qn, qr, row, tf, tc, nt, window, meta, st):
-        """Prompt portions: every sequence's visible latents up-projected into per-head keys and values -> launches."""
-        L, dt, dev, tdt = self.L, self.dt, self.dev, self.m.dtype
-        H, dn, dr, dv, R, n = a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, meta.n
-        src, launches = meta.extra.get(("rows", window)), 2
-        if src is not None:
-            ca, kra = torch.empty(len(src), R, dtype=tdt, device=dev), torch.empty(len(src), dr, dtype=tdt, device=dev)
-            _lib.lm_check(L.ao_lm_latent_rows_gather(_p(src), len(src), _p(c), _p(kr), _p(cache.c), _p(cache.kr), dt, R, dr, _p(ca),
-                                                     _p(kra), st), "latent_rows_gather")
-            c, kr, launches = ca, kra, 3
-        kv = torch.mm(c, lay.ukv.t())                                                  # [rows][H dn | H dv]
-        ld = H * (dn + dv)
-        _lib.lm_check(L.ao_lm_window_latent_attention_expanded(
-            _p(qn), _p(qr), _p(kv), ld, kv.data_ptr() + kv.element_size() * H * dn, ld, _p(kr), dt, _p(meta.pos), _p(tf), _p(tc),
-            _p(meta.extra[("key0", window)]), nt, n, H, dn, dr, dv, a.scale, window, None, None, _p(row), row.shape[1], st),
-            "window_latent_attention_expanded")
-        return launches
-
-    def _bmm_f32(self, a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-        """[b][n][K] x [b][K][M] -> fp32 [b][n][M]."""
-        return torch.bmm(a, w, out_dtype=torch.float32) if a.dtype == torch.bfloat16 else torch.bmm(a, w)
 
     def _logits_dev(self, x, d_rows, k, out=None):
         m, cfg = self.m, self.cfg

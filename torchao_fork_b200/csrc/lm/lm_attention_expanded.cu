@@ -31,7 +31,7 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
                             const int32_t* __restrict__ tile_count, const int32_t* __restrict__ tile_kv_row, int64_t n, int H,
                             int dn, int dr, float scale, const __nv_bfloat16* __restrict__ sink,
                             const float* __restrict__ gate, __nv_bfloat16* __restrict__ out, int64_t ldk, int64_t ldv, int window,
-                            int64_t ld_out) {
+                            int64_t ld_out, const float* __restrict__ gate_rows, int64_t ld_gate) {
   using T = __nv_bfloat16;
   constexpr int DV = 16 * NV;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -229,7 +229,12 @@ latent_attn_expanded_kernel(const __nv_bfloat16* __restrict__ qn, const float* _
     T* dst = out + t * ld_out + (int64_t)h * DV + 2 * t4;
 #pragma unroll
     for (int i = 0; i < 2 * NV; ++i) {
-      const float y0 = o[i][2 * half] * k, y1 = o[i][2 * half + 1] * k;
+      float y0 = o[i][2 * half] * k, y1 = o[i][2 * half + 1] * k;
+      if (gate_rows) {   // a gate per output element, as a logit
+        const float* gl = gate_rows + t * ld_gate + (int64_t)h * DV + 2 * t4 + i * 8;
+        y0 /= 1.f + __expf(-gl[0]);
+        y1 /= 1.f + __expf(-gl[1]);
+      }
       if (pairs) {
         *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(y0, y1);
       } else {   // rows of odd length: every other row starts on an odd element
@@ -250,7 +255,8 @@ template <int NV>
 int launch_expanded(const void* qn, const float* qr, const void* kx, const void* vx, const void* kr_cache, int64_t S,
                     const int32_t* slot, const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count,
                     const int32_t* tile_kv_row, int n_tiles, int64_t n, int H, int dn, int dr, float scale, const void* sink,
-                    const float* gate, void* out, int64_t ldk, int64_t ldv, int window, int64_t ld_out, cudaStream_t st) {
+                    const float* gate, void* out, int64_t ldk, int64_t ldv, int window, int64_t ld_out, const float* gate_rows,
+                    int64_t ld_gate, cudaStream_t st) {
   using T = __nv_bfloat16;
   const size_t smem = ((size_t)kPM * (dn + 2 * dr + kPad) + (size_t)kPN * (dn + dr + kPad) + (size_t)kPN * (16 * NV + kPad)) * 2;
   auto kern = latent_attn_expanded_kernel<NV>;
@@ -265,7 +271,7 @@ int launch_expanded(const void* qn, const float* qr, const void* kx, const void*
   kern<<<grid, kPWarps * 32, smem, st>>>(static_cast<const T*>(qn), qr, static_cast<const T*>(kx), static_cast<const T*>(vx),
                                          static_cast<const T*>(kr_cache), S, slot, pos, tile_first, tile_count, tile_kv_row, n, H,
                                          dn, dr, scale, static_cast<const T*>(sink), gate, static_cast<T*>(out), ldk, ldv, window,
-                                         ld_out);
+                                         ld_out, gate_rows, ld_gate);
   return lm_launch_status();
 }
 
@@ -281,11 +287,11 @@ static int dispatch_expanded(const void* qn, const float* qr, const void* kx, co
                              const int32_t* slot, const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count,
                              const int32_t* tile_kv_row, int n_tiles, int64_t n, int H, int dn, int dr, int dv, float scale,
                              const void* sink, const float* gate, void* out, int64_t ldk, int64_t ldv, int window, int64_t ld_out,
-                             cudaStream_t st) {
+                             const float* gate_rows, int64_t ld_gate, cudaStream_t st) {
 #define LM_XP(NV)                                                                                                                  \
   case NV:                                                                                                                         \
     return launch_expanded<NV>(qn, qr, kx, vx, kr, S, slot, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, scale, \
-                               sink, gate, out, ldk, ldv, window, ld_out, st);
+                               sink, gate, out, ldk, ldv, window, ld_out, gate_rows, ld_gate, st);
   switch (dv / 16) { LM_XP(1) LM_XP(2) LM_XP(3) LM_XP(4) LM_XP(5) LM_XP(6) LM_XP(7) LM_XP(8) }
 #undef LM_XP
   return AO_B200_ERR_UNSUPPORTED;
@@ -301,7 +307,32 @@ extern "C" int ao_lm_latent_attention_expanded(const void* qn, const float* qr, 
   LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && H <= 65535 && S > 0);
   if (!expanded_ok(dt, dn, dr, dv)) return AO_B200_ERR_UNSUPPORTED;
   return dispatch_expanded(qn, qr, kx, vx, kr_cache, S, slot, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, dv, scale,
-                           sink, gate, out, (int64_t)H * dn, (int64_t)H * dv, 0x7fffffff, (int64_t)H * dv, lm_stream(stream));
+                           sink, gate, out, (int64_t)H * dn, (int64_t)H * dv, 0x7fffffff, (int64_t)H * dv, nullptr, 0, lm_stream(stream));
+}
+
+static int expanded_rows(const void* qn, const float* qr, const void* kx, int64_t ldk, const void* vx, int64_t ldv, const void* kr, int dt,
+                         const int32_t* pos, const int32_t* tile_first, const int32_t* tile_count, const int32_t* tile_kv_row, int n_tiles,
+                         int64_t n, int H, int dn, int dr, int dv, float scale, int window, const void* sink, const float* gate,
+                         const float* gate_rows, int64_t ld_gate, void* out, int64_t ld_out, void* stream) {
+  LM_CHECK_ARG(qn && kx && vx && pos && tile_first && tile_count && tile_kv_row && out && ((qr && kr) || dr == 0));
+  LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && H <= 65535 && window > 0 && ldk >= (int64_t)H * dn && ldv >= (int64_t)H * dv && ld_out >= (int64_t)H * dv);
+  LM_CHECK_ARG(!gate_rows || ld_gate >= (int64_t)H * dv);
+  if (!expanded_ok(dt, dn, dr, dv)) return AO_B200_ERR_UNSUPPORTED;
+  // 16-byte copies of queries, keys and values; the result is stored in pairs when its rows allow it
+  LM_CHECK_ARG(ldk % 8 == 0 && ldv % 8 == 0 && reinterpret_cast<uintptr_t>(qn) % 16 == 0 && reinterpret_cast<uintptr_t>(qr) % 16 == 0 &&
+               reinterpret_cast<uintptr_t>(kx) % 16 == 0 && reinterpret_cast<uintptr_t>(vx) % 16 == 0 &&
+               reinterpret_cast<uintptr_t>(kr) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 4 == 0);
+  return dispatch_expanded(qn, qr, kx, vx, kr, 0, nullptr, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, dv, scale,
+                           sink, gate, out, ldk, ldv, window, ld_out, gate_rows, ld_gate, lm_stream(stream));
+}
+
+extern "C" int ao_lm_gated_latent_attention_expanded(const void* qn, const float* qr, const void* kx, int64_t ldk, const void* vx,
+                                                     int64_t ldv, const void* kr, int dt, const int32_t* pos, const int32_t* tile_first,
+                                                     const int32_t* tile_count, const int32_t* tile_kv_row, int n_tiles, int64_t n, int H,
+                                                     int dn, int dr, int dv, float scale, int window, const void* sink,
+                                                     const float* gate_rows, int64_t ld_gate, void* out, int64_t ld_out, void* stream) {
+  return expanded_rows(qn, qr, kx, ldk, vx, ldv, kr, dt, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, dv, scale, window,
+                       sink, nullptr, gate_rows, ld_gate, out, ld_out, stream);
 }
 
 extern "C" int ao_lm_window_latent_attention_expanded(const void* qn, const float* qr, const void* kx, int64_t ldk, const void* vx,
@@ -310,13 +341,6 @@ extern "C" int ao_lm_window_latent_attention_expanded(const void* qn, const floa
                                                       const int32_t* tile_kv_row, int n_tiles, int64_t n, int H, int dn, int dr,
                                                       int dv, float scale, int window, const void* sink, const float* gate,
                                                       void* out, int64_t ld_out, void* stream) {
-  LM_CHECK_ARG(qn && kx && vx && pos && tile_first && tile_count && tile_kv_row && out && ((qr && kr) || dr == 0));
-  LM_CHECK_ARG(n > 0 && n_tiles > 0 && H > 0 && H <= 65535 && window > 0 && ldk >= (int64_t)H * dn && ldv >= (int64_t)H * dv && ld_out >= (int64_t)H * dv);
-  if (!expanded_ok(dt, dn, dr, dv)) return AO_B200_ERR_UNSUPPORTED;
-  // 16-byte copies of queries, keys and values; the result is stored in pairs when its rows allow it
-  LM_CHECK_ARG(ldk % 8 == 0 && ldv % 8 == 0 && reinterpret_cast<uintptr_t>(qn) % 16 == 0 && reinterpret_cast<uintptr_t>(qr) % 16 == 0 &&
-               reinterpret_cast<uintptr_t>(kx) % 16 == 0 && reinterpret_cast<uintptr_t>(vx) % 16 == 0 &&
-               reinterpret_cast<uintptr_t>(kr) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 4 == 0);
-  return dispatch_expanded(qn, qr, kx, vx, kr, 0, nullptr, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, dv, scale,
-                           sink, gate, out, ldk, ldv, window, ld_out, lm_stream(stream));
+  return expanded_rows(qn, qr, kx, ldk, vx, ldv, kr, dt, pos, tile_first, tile_count, tile_kv_row, n_tiles, n, H, dn, dr, dv, scale, window,
+                       sink, gate, nullptr, 0, out, ld_out, stream);
 }

@@ -35,13 +35,6 @@ __device__ __forceinline__ float dot4(const float4& x, const float4& y, float ac
   return fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, acc))));
 }
 
-__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16),
-                     __uint_as_float(u.y & 0xFFFF0000u));
-}
-
 struct DeltaArgs {
   const float* qk;               // [n][2][G][dp]: unit queries (scaled), unit keys; zeros beyond d
   const float* v;                // [n][H dv]

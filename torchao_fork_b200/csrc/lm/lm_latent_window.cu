@@ -1,8 +1,11 @@
-// Latent attention whose queries also come from a latent, under a sliding window: what happens between its projections.
+// Latent attention whose queries also come from a latent, under a sliding window or over a full cache: what happens between its projections.
 //     ao_lm_latent_low_prep     projection row -> normed query latent, normed key/value latent, rotated shared key part
+//                               (_store: also into a cache that never wraps, which saves the append launch)
 //     ao_lm_latent_query_prep   up-projected queries -> unrotated parts (head-major) and rotated parts
 //     ao_lm_latent_rows_gather  the rows a step's queries can see, contiguous per sequence: window rows that earlier steps
 //                               left in the ring, then the step's own
+//     ao_lm_latent_value_up     weighted latents of few rows -> heads, times the sigmoid of an element-wise gate
+//     ao_lm_sigmoid_gate_rows   the gate alone, in place (many rows: a library product made the heads)
 // The step's latents stay in step buffers until its attention has run (ao_lm_ring_append then stores them): a long portion
 // would otherwise overwrite ring rows that its first queries still need.  Norms and angles are fp32.
 #include "lm_common.cuh"
@@ -11,42 +14,84 @@ using namespace lm;
 
 namespace {
 
-// out[0 .. count) = src / sqrt(mean(src^2) + eps) * weight by the whole block
-template <typename T>
-__device__ __forceinline__ void norm_part(const float* __restrict__ src, int count, const T* __restrict__ weight, float eps,
-                                          T* __restrict__ out, float* scratch) {
+template <bool VEC>
+__device__ __forceinline__ float part_squares(const float* __restrict__ src, int count) {
   float ss = 0.f;
-  for (int i = threadIdx.x; i < count; i += blockDim.x) ss = fmaf(src[i], src[i], ss);
-  const float k = 1.f / sqrtf(block_sum(ss, scratch) / (float)count + eps);
-  for (int i = threadIdx.x; i < count; i += blockDim.x) stf(out + i, src[i] * k * ldf(weight + i));
+  if (VEC) {
+    for (int i = threadIdx.x * 4; i < count; i += blockDim.x * 4) {
+      const float4 v = ld4(src + i);
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+  } else {
+    for (int i = threadIdx.x; i < count; i += blockDim.x) ss = fmaf(src[i], src[i], ss);
+  }
+  return ss;
+}
+// out (and also, unless it is null) = src * k * weight
+template <typename T, bool VEC>
+__device__ __forceinline__ void scale_part(const float* __restrict__ src, int count, float k, const T* __restrict__ weight, T* __restrict__ out,
+                                           T* __restrict__ also) {
+  if (VEC) {
+    for (int i = threadIdx.x * 4; i < count; i += blockDim.x * 4) {
+      float4 v = ld4(src + i);
+      const float4 g = ld4(weight + i);
+      v.x *= k * g.x, v.y *= k * g.y, v.z *= k * g.z, v.w *= k * g.w;
+      st4(out + i, v);
+      if (also) st4(also + i, v);
+    }
+  } else {
+    for (int i = threadIdx.x; i < count; i += blockDim.x) {
+      const float v = src[i] * k * ldf(weight + i);
+      stf(out + i, v);
+      if (also) stf(also + i, v);
+    }
+  }
 }
 
-template <typename T>
+// One CTA per row.  The two norms' sums meet in one reduction (the row is read again from L1 for the output).  With c_cache the
+// latent and the rotated part also go to row pos[t] of the slot (a cache that never wraps).
+template <typename T, bool VEC>
 __global__ void latent_low_prep_kernel(const float* __restrict__ proj, int64_t ld, int64_t q_off, int Rq, int64_t kv_off, int R, int dr,
                                        const T* __restrict__ q_norm, const T* __restrict__ c_norm, float eps, int rot_dims,
                                        const float* __restrict__ inv_freq, float amp, const int32_t* __restrict__ pos,
-                                       T* __restrict__ cq, T* __restrict__ c, T* __restrict__ kr) {
-  __shared__ float scratch[33];
+                                       const int32_t* __restrict__ slot, int64_t S, T* __restrict__ cq, T* __restrict__ c, T* __restrict__ kr,
+                                       T* __restrict__ c_cache, T* __restrict__ kr_cache) {
+  __shared__ float2 sums[32];
   const int64_t t = blockIdx.x;
   const float* row = proj + t * ld;
-  norm_part(row + q_off, Rq, q_norm, eps, cq + t * Rq, scratch);
-  norm_part(row + kv_off, R, c_norm, eps, c + t * R, scratch);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const float* src = row + kv_off + R;
-  T* dst = kr + t * dr;
-  const float p = (float)pos[t];
   const int half = rot_dims / 2;
+  const int p = pos[t];
+  const int64_t at = c_cache ? (int64_t)slot[t] * S + p : 0;
+  float sq = warp_sum(part_squares<VEC>(row + q_off, Rq)), sc = warp_sum(part_squares<VEC>(row + kv_off, R));
+  if (lane == 0) sums[warp] = make_float2(sq, sc);
+  // the shared key part meanwhile
+  T* dst = kr + t * dr;
+  T* also = kr_cache ? kr_cache + at * dr : nullptr;
   for (int i = threadIdx.x; i < dr - half; i += blockDim.x) {
     if (i < half) {
       float sn, cs;
-      sincosf(p * inv_freq[i], &sn, &cs);
+      sincosf((float)p * inv_freq[i], &sn, &cs);
       sn *= amp, cs *= amp;
       const float u = src[2 * i], v = src[2 * i + 1];
-      stf(dst + 2 * i, u * cs - v * sn);
-      stf(dst + 2 * i + 1, v * cs + u * sn);
+      const float a = u * cs - v * sn, b = v * cs + u * sn;
+      stf(dst + 2 * i, a);
+      stf(dst + 2 * i + 1, b);
+      if (also) {
+        stf(also + 2 * i, a);
+        stf(also + 2 * i + 1, b);
+      }
     } else {
       stf(dst + half + i, src[half + i]);     // coordinates from rot_dims on pass
+      if (also) stf(also + half + i, src[half + i]);
     }
   }
+  __syncthreads();
+  const float2 mine = lane < nw ? sums[lane] : make_float2(0.f, 0.f);
+  sq = warp_sum(mine.x), sc = warp_sum(mine.y);
+  scale_part<T, VEC>(row + q_off, Rq, 1.f / sqrtf(sq / (float)Rq + eps), q_norm, cq + t * Rq, nullptr);
+  scale_part<T, VEC>(row + kv_off, R, 1.f / sqrtf(sc / (float)R + eps), c_norm, c + t * R, c_cache ? c_cache + at * R : nullptr);
 }
 
 // q [n][H][dn + dr] -> qn[h][t][dn] in T, qr[t][h][dr] rotated, fp32.  A row may be shared by several CTAs.
@@ -102,17 +147,81 @@ __global__ void latent_rows_gather_kernel(const int32_t* __restrict__ src, const
   for (int e = threadIdx.x; e < dr; e += blockDim.x) out_kr[i * dr + e] = b[e];
 }
 
+// out[t][h dv + j] = sigmoid(gate[t][h dv + j]) * sum_r uv[h][j][r] * olat[t][h][r].  One CTA = one row x one head x kUpOut
+// outputs; a warp makes four of them at a time from one pass over their weight rows.
+constexpr int kUpWarps = 8, kUpPer = 4, kUpOut = kUpWarps * kUpPer;
+template <typename T>
+__global__ void __launch_bounds__(kUpWarps * 32) latent_value_up_kernel(const T* __restrict__ olat, const T* __restrict__ uv, int H, int R,
+                                                                        int dv, const float* __restrict__ gate, int64_t ld_gate, bool vec,
+                                                                        T* __restrict__ out, int64_t ld_out) {
+  extern __shared__ __align__(16) float xs[];
+  const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int64_t t = blockIdx.z;
+  const int j0 = blockIdx.x * kUpOut + warp * kUpPer, nr = min(kUpPer, dv - j0);
+  const T* rows[kUpPer];
+  const float* x[kUpPer];
+#pragma unroll
+  for (int i = 0; i < kUpPer; ++i) rows[i] = uv + ((int64_t)h * dv + (i < nr ? j0 + i : 0)) * R, x[i] = xs;
+  stage_f32(olat + (t * H + h) * R, xs, R);
+  __syncthreads();
+  if (nr <= 0) return;
+  float acc[kUpPer];
+  if constexpr (sizeof(T) == 2) {
+    if (vec) {
+      warp_dot_rows<kUpPer, 2>(rows, x, nr, R, lane, acc);
+    } else {
+#pragma unroll
+      for (int i = 0; i < kUpPer; ++i) acc[i] = warp_dot(rows[i], xs, R, lane, false);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < kUpPer; ++i) acc[i] = warp_dot(rows[i], xs, R, lane, vec);
+  }
+  if (lane < nr) {
+    float v = acc[0];
+#pragma unroll
+    for (int i = 1; i < kUpPer; ++i)
+      if (lane == i) v = acc[i];
+    const int64_t col = (int64_t)h * dv + j0 + lane;
+    if (gate) v = v / (1.f + expf(-gate[t * ld_gate + col]));
+    stf(out + t * ld_out + col, v);
+  }
+}
+
+template <typename T>
+__global__ void sigmoid_gate_rows_kernel(const float* __restrict__ gate, int64_t ld_gate, int64_t cols, T* y, int64_t ld) {
+  const int64_t t = blockIdx.x;
+  for (int64_t c = (int64_t)blockIdx.y * blockDim.x + threadIdx.x; c < cols; c += (int64_t)gridDim.y * blockDim.x)
+    stf(y + t * ld + c, ldf(y + t * ld + c) / (1.f + expf(-gate[t * ld_gate + c])));
+}
+
 }  // namespace
+
+extern "C" int ao_lm_latent_low_prep_store(const float* proj, int64_t ld, int64_t n, int64_t q_off, int Rq, int64_t kv_off, int R, int dr,
+                                           const void* q_norm, const void* c_norm, int dt, float eps, int rot_dims, const float* inv_freq,
+                                           float amp, const int32_t* pos, const int32_t* slot, int64_t S, void* cq, void* c, void* kr,
+                                           void* c_cache, void* kr_cache, void* stream) {
+  LM_CHECK_ARG(proj && q_norm && c_norm && pos && cq && c && (kr || dr == 0) && n > 0 && Rq > 0 && R > 0 && dr >= 0);
+  LM_CHECK_ARG(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq));
+  LM_CHECK_ARG(!c_cache || (slot && S > 0 && (kr_cache || dr == 0)));
+  LM_DISPATCH(dt, {
+    auto on = [](const void* p, size_t bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
+    const size_t four = 4 * sizeof(T);
+    const bool vec = ld % 4 == 0 && q_off % 4 == 0 && kv_off % 4 == 0 && Rq % 4 == 0 && R % 4 == 0 && on(proj, 16) && on(q_norm, four) &&
+                     on(c_norm, four) && on(cq, four) && on(c, four) && on(c_cache, four);
+    auto kern = vec ? latent_low_prep_kernel<T, true> : latent_low_prep_kernel<T, false>;
+    kern<<<(unsigned)n, n < 296 && !vec ? 512 : n < 296 ? 256 : 128, 0, lm_stream(stream)>>>(
+        proj, ld, q_off, Rq, kv_off, R, dr, static_cast<const T*>(q_norm), static_cast<const T*>(c_norm), eps, rot_dims, inv_freq, amp, pos,
+        slot, S, static_cast<T*>(cq), static_cast<T*>(c), static_cast<T*>(kr), static_cast<T*>(c_cache), static_cast<T*>(kr_cache));
+  });
+  return lm_launch_status();
+}
 
 extern "C" int ao_lm_latent_low_prep(const float* proj, int64_t ld, int64_t n, int64_t q_off, int Rq, int64_t kv_off, int R, int dr,
                                      const void* q_norm, const void* c_norm, int dt, float eps, int rot_dims, const float* inv_freq,
                                      float amp, const int32_t* pos, void* cq, void* c, void* kr, void* stream) {
-  LM_CHECK_ARG(proj && q_norm && c_norm && pos && cq && c && (kr || dr == 0) && n > 0 && Rq > 0 && R > 0 && dr >= 0);
-  LM_CHECK_ARG(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq));
-  LM_DISPATCH(dt, latent_low_prep_kernel<T><<<(unsigned)n, n < 296 ? 512 : 128, 0, lm_stream(stream)>>>(
-                      proj, ld, q_off, Rq, kv_off, R, dr, static_cast<const T*>(q_norm), static_cast<const T*>(c_norm), eps, rot_dims,
-                      inv_freq, amp, pos, static_cast<T*>(cq), static_cast<T*>(c), static_cast<T*>(kr)));
-  return lm_launch_status();
+  return ao_lm_latent_low_prep_store(proj, ld, n, q_off, Rq, kv_off, R, dr, q_norm, c_norm, dt, eps, rot_dims, inv_freq, amp, pos, nullptr, 0,
+                                     cq, c, kr, nullptr, nullptr, stream);
 }
 
 extern "C" int ao_lm_latent_query_prep(const float* q, int64_t n, int H, int dn, int dr, int dt, int rot_dims, const float* inv_freq,
@@ -133,5 +242,27 @@ extern "C" int ao_lm_latent_rows_gather(const int32_t* src, int64_t rows, const 
   LM_DISPATCH(dt, latent_rows_gather_kernel<T><<<(unsigned)rows, 64, 0, lm_stream(stream)>>>(
                       src, static_cast<const T*>(c), static_cast<const T*>(kr), static_cast<const T*>(ring_c),
                       static_cast<const T*>(ring_kr), R, dr, static_cast<T*>(out_c), static_cast<T*>(out_kr)));
+  return lm_launch_status();
+}
+
+extern "C" int ao_lm_latent_value_up(const void* olat, const void* uv, int dt, int64_t n, int H, int R, int dv, const float* gate,
+                                     int64_t ld_gate, void* out, int64_t ld_out, void* stream) {
+  LM_CHECK_ARG(olat && uv && out && n > 0 && n <= 65535 && H > 0 && H <= 65535 && R > 0 && dv > 0 && ld_out >= (int64_t)H * dv &&
+               (!gate || ld_gate >= (int64_t)H * dv));
+  if ((size_t)R * sizeof(float) > 48 * 1024) return AO_B200_ERR_UNSUPPORTED;
+  LM_DISPATCH(dt, latent_value_up_kernel<T><<<dim3((unsigned)((dv + kUpOut - 1) / kUpOut), (unsigned)H, (unsigned)n), kUpWarps * 32,
+                                              (size_t)R * sizeof(float), lm_stream(stream)>>>(
+                      static_cast<const T*>(olat), static_cast<const T*>(uv), H, R, dv, gate, ld_gate, rows_vectorizable<T>(uv, R),
+                      static_cast<T*>(out), ld_out));
+  return lm_launch_status();
+}
+
+extern "C" int ao_lm_sigmoid_gate_rows(const float* gate, int64_t ld_gate, int64_t n, int64_t cols, void* y, int64_t ld, int dt,
+                                       void* stream) {
+  LM_CHECK_ARG(gate && y && n > 0 && cols > 0 && ld >= cols && ld_gate >= cols);
+  int64_t parts = (cols + 511) / 512;
+  if (parts > 64) parts = 64;
+  LM_DISPATCH(dt, sigmoid_gate_rows_kernel<T><<<dim3((unsigned)n, (unsigned)parts), 256, 0, lm_stream(stream)>>>(
+                      gate, ld_gate, cols, static_cast<T*>(y), ld));
   return lm_launch_status();
 }

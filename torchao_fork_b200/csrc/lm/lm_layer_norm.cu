@@ -2,6 +2,8 @@
 // a constant times each sublayer's result: the residual add fused with the next sublayer's norm; rotary positions applied
 // in place to an fp32 projection (both pairings of coordinates); the inputs of a time-mixing layer that blends every row
 // with its predecessor through several learned vectors at once; element-wise activations between two projections.
+#include <type_traits>
+
 #include "lm_common.cuh"
 
 using namespace lm;
@@ -86,23 +88,29 @@ __global__ void token_shift_mix_kernel(const float* __restrict__ h, const T* __r
   }
 }
 
-template <typename TI, typename TO>
+__device__ __forceinline__ float unary(float z, int kind, float param) {
+  if (kind == 0) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  }
+  return kind == 1 ? tanhf(z) : param * tanhf(z / param);
+}
+
+// VEC: cols is a multiple of four and both rows start on aligned groups of four
+template <typename TI, typename TO, bool VEC>
 __global__ void unary_rows_kernel(const TI* in, int64_t cols, int kind, float param, const float* __restrict__ row_scale,
                                   int64_t ld_scale, TO* out) {
   const int64_t t = blockIdx.x;
   const float k = row_scale ? row_scale[t * ld_scale] : 1.f;
-  for (int64_t c = blockIdx.y * blockDim.x + threadIdx.x; c < cols; c += (int64_t)gridDim.y * blockDim.x) {
-    const float z = ldf(in + t * cols + c);
-    float v;
-    if (kind == 0) {
-      const float r = fmaxf(z, 0.f);
-      v = r * r;
-    } else if (kind == 1) {
-      v = tanhf(z);
-    } else {
-      v = param * tanhf(z / param);
+  const int64_t i0 = (int64_t)blockIdx.y * blockDim.x + threadIdx.x, step = (int64_t)gridDim.y * blockDim.x;
+  if (VEC) {
+    for (int64_t c = i0 * 4; c < cols; c += step * 4) {
+      const float4 z = ld4(in + t * cols + c);
+      st4(out + t * cols + c, make_float4(unary(z.x, kind, param) * k, unary(z.y, kind, param) * k, unary(z.z, kind, param) * k,
+                                          unary(z.w, kind, param) * k));
     }
-    stf(out + t * cols + c, v * k);
+  } else {
+    for (int64_t c = i0; c < cols; c += step) stf(out + t * cols + c, unary(ldf(in + t * cols + c), kind, param) * k);
   }
 }
 
@@ -171,19 +179,25 @@ extern "C" int ao_lm_token_shift_mix(const float* h, const void* mu, int n_mix, 
 extern "C" int ao_lm_unary_rows(const void* in, int in_dt, int64_t n, int64_t cols, int kind, float param, const float* row_scale,
                                 int64_t ld_scale, void* out, int out_dt, void* stream) {
   LM_CHECK_ARG(in && out && n > 0 && cols > 0 && kind >= 0 && kind <= 2 && (kind != 2 || param > 0.f));
+  auto on = [](const void* p, int dt) { return reinterpret_cast<uintptr_t>(p) % (dt == AO_LM_BF16 ? 8 : 16) == 0; };
+  const bool vec = cols % 4 == 0 && on(in, in_dt) && on(out, out_dt);
   const cudaStream_t st = lm_stream(stream);
-  const unsigned th = threads_for(cols);
-  const dim3 grid = row_grid(n, cols, th);
+  const int64_t items = vec ? cols / 4 : cols;
+  const unsigned th = threads_for(items);
+  const int64_t parts = (items + 2 * th - 1) / (2 * th);         // about two accesses per thread
+  const dim3 grid((unsigned)n, (unsigned)(parts > 64 ? 64 : parts));
+  auto run = [&](auto* i, auto* o) {
+    using TI = std::remove_const_t<std::remove_pointer_t<decltype(i)>>;
+    using TO = std::remove_pointer_t<decltype(o)>;
+    if (vec) unary_rows_kernel<TI, TO, true><<<grid, th, 0, st>>>(i, cols, kind, param, row_scale, ld_scale, o);
+    else unary_rows_kernel<TI, TO, false><<<grid, th, 0, st>>>(i, cols, kind, param, row_scale, ld_scale, o);
+  };
   if (in_dt == AO_LM_F32 && out_dt == AO_LM_F32)
-    unary_rows_kernel<float, float><<<grid, th, 0, st>>>(static_cast<const float*>(in), cols, kind, param, row_scale, ld_scale,
-                                                                static_cast<float*>(out));
+    run(static_cast<const float*>(in), static_cast<float*>(out));
   else if (in_dt == AO_LM_F32 && out_dt == AO_LM_BF16)
-    unary_rows_kernel<float, __nv_bfloat16><<<grid, th, 0, st>>>(static_cast<const float*>(in), cols, kind, param, row_scale,
-                                                                        ld_scale, static_cast<__nv_bfloat16*>(out));
+    run(static_cast<const float*>(in), static_cast<__nv_bfloat16*>(out));
   else if (in_dt == AO_LM_BF16 && out_dt == AO_LM_BF16)
-    unary_rows_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, th, 0, st>>>(static_cast<const __nv_bfloat16*>(in), cols, kind,
-                                                                                param, row_scale, ld_scale,
-                                                                                static_cast<__nv_bfloat16*>(out));
+    run(static_cast<const __nv_bfloat16*>(in), static_cast<__nv_bfloat16*>(out));
   else
     return AO_B200_ERR_INVALID_ARG;
   return lm_launch_status();

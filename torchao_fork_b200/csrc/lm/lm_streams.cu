@@ -115,20 +115,8 @@ __global__ void __launch_bounds__(1024) streams_update_kernel(float* __restrict_
   }
 }
 
-
 // ---- the same two kernels for widths that are multiples of 4: 16-byte loads and stores, the stream count a
 // compile-time constant (no predicated loops)
-__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ void st4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16),
-                     __uint_as_float(u.y & 0xFFFF0000u));
-}
-__device__ __forceinline__ void st4(__nv_bfloat16* p, const float4& v) {
-  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-}
 
 template <typename T, int S>
 __global__ void __launch_bounds__(512) streams_norm_vec_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows,
