@@ -14,6 +14,7 @@ streams them from HBM (no L2 flush needed).  Prints ONE JSON line (see the task 
 --impl reference times that CPU path alone (rank 0 only).  N > 1: tensor parallel (tp.py), strong scaling.
 """
 import argparse
+import importlib
 import json
 import os
 import statistics
@@ -586,17 +587,18 @@ def run_b200(args):
         os._exit(0)
 
 
+LAYER_WORKLOADS = [f + "-layers" for f in ("bitipel", "tadolix", "rutusun", "fedipel", "rigalorn", "sozanex")]
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=200)  # reference: 200 new tokens per sample (generate.py:264)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--workload", default="llama3-8b-int4", choices=sorted(WORKLOADS) + ["bitipel-layers", "tadolix-layers", "rutusun-layers", "fedipel-layers", "rigalorn-layers"],
-                    help="bitipel-layers / tadolix-layers / rutusun-layers / fedipel-layers / rigalorn-layers: prefill / decode of that family's layers at real sizes "
-                         "beside the closest other family at equal size (benchmarks/bitipel_bench.py, tadolix_bench.py, rutusun_bench.py, "
-                         "fedipel_bench.py, rigalorn_bench.py; their own JSON line, not "
-                         "the headline metric)")
+    ap.add_argument("--workload", default="llama3-8b-int4", choices=sorted(WORKLOADS) + LAYER_WORKLOADS,
+                    help="<family>-layers: prefill / decode of that family's layers at real sizes beside the closest other family at "
+                         "equal size (benchmarks/<family>_bench.py; their own JSON line, not the headline metric)")
     ap.add_argument("--batch-size", type=int, default=1)
     ap.add_argument("--temperature", type=float, default=0.8)
     ap.add_argument("--top-k", type=int, default=200)
@@ -604,30 +606,9 @@ def main():
     ap.add_argument("--cpu-budget-s", type=float, default=25.0, help="reference arm: stop timing tokens after this many seconds")
     ap.add_argument("--no-reference-gpu", action="store_true")
     args = ap.parse_args()
-    if args.workload == "bitipel-layers":
-        assert args.impl == "b200" and args.gpus == 1, "bitipel-layers is a one-GPU measurement of this repo's kernels"
-        from benchmarks import bitipel_bench
-        emit(bitipel_bench.run())
-        return
-    if args.workload == "tadolix-layers":
-        assert args.impl == "b200" and args.gpus == 1, "tadolix-layers is a one-GPU measurement of this repo's kernels"
-        from benchmarks import tadolix_bench
-        emit(tadolix_bench.run())
-        return
-    if args.workload == "fedipel-layers":
-        assert args.impl == "b200" and args.gpus == 1, "fedipel-layers is a one-GPU measurement of this repo's kernels"
-        from benchmarks import fedipel_bench
-        emit(fedipel_bench.run())
-        return
-    if args.workload == "rigalorn-layers":
-        assert args.impl == "b200" and args.gpus == 1, "rigalorn-layers is a one-GPU measurement of this repo's kernels"
-        from benchmarks import rigalorn_bench
-        emit(rigalorn_bench.run())
-        return
-    if args.workload == "rutusun-layers":
-        assert args.impl == "b200" and args.gpus == 1, "rutusun-layers is a one-GPU measurement of this repo's kernels"
-        from benchmarks import rutusun_bench
-        emit(rutusun_bench.run())
+    if args.workload in LAYER_WORKLOADS:
+        assert args.impl == "b200" and args.gpus == 1, f"{args.workload} is a one-GPU measurement of this repo's kernels"
+        emit(importlib.import_module("benchmarks." + args.workload.replace("-layers", "_bench")).run())
         return
     if args.impl == "reference":
         run_reference(args)

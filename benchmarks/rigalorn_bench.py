@@ -26,14 +26,15 @@ FP32_TFLOPS = 148 * 128 * 2 * 1.9e9 / 1e12
 BF16, F32 = 0, 1
 
 
-def model_numbers(names, prompt_len, decode_ctx, decode_steps):
-    """prefill tokens/s of a prompt and decode tokens/s (batch 1, CUDA graph) for every named configuration."""
+def model_numbers(names, prompt_len, decode_ctx, decode_steps, make=None):
+    """prefill tokens/s of a prompt and decode tokens/s (batch 1, CUDA graph) for every named configuration; make: name -> a
+    function that builds the model, for configurations that the registry does not name."""
     from torchao_fork_b200._models import registry
     from torchao_fork_b200._models.llama.generate import Generator, prefill
     dev = torch.device("cuda")
     out = {}
     for nm in names:
-        model = registry.random_init(nm, dev, torch.bfloat16)
+        model = make[nm]() if make and nm in make else registry.random_init(nm, dev, torch.bfloat16)
         S = max(prompt_len, decode_ctx + decode_steps + 8)
         gen = Generator(model, 1, S, temperature=0.0, top_k=None)
         prompt = torch.randint(0, model.config.vocab_size, (1, prompt_len), device=dev)
@@ -62,15 +63,19 @@ class Bench:
     """Kernels alone at one configuration's layer shapes."""
 
     def __init__(self, name, prompt_len, decode_ctx):
-        from torchao_fork_b200 import _lib
         from torchao_fork_b200._models.rigalorn import rigalorn_configs
+        self.setup(rigalorn_configs[name](), prompt_len, decode_ctx)
+        self.delta = self.by["delta"].mixer
+
+    def setup(self, cfg, prompt_len, decode_ctx):
+        from torchao_fork_b200 import _lib
         self.lib, self.L = _lib, _lib.lm()
         self.hbm, self.tf, self.src = peaks()
         self.dev = torch.device("cuda")
         self.st = torch.cuda.current_stream().cuda_stream
-        self.cfg = rigalorn_configs[name]()
-        by = {la.type: la for la in self.cfg.layers}
-        self.att, self.delta, self.lat = by["attention"].mixer, by["delta"].mixer, by["latent_attention"].mixer
+        self.cfg = cfg
+        self.by = {la.type: la for la in cfg.layers}
+        self.att, self.lat = self.by["attention"].mixer, self.by["latent_attention"].mixer
         self.ff, self.W, self.n, self.ctx = self.cfg.layers[0].ff, self.cfg.width, prompt_len, decode_ctx
         self.flush = torch.zeros(64 << 20, dtype=torch.float32, device=self.dev)
         pos = np.arange(prompt_len)
