@@ -552,12 +552,23 @@ AO_B200_API int ao_lm_gated_latent_attention_expanded(const void* qn, const floa
                                                       const int32_t* tile_count, const int32_t* tile_kv_row, int n_tiles, int64_t n, int H,
                                                       int dn, int dr, int dv, float scale, int window, const void* sink,
                                                       const float* gate_rows, int64_t ld_gate, void* out, int64_t ld_out, void* stream);
+/* The folded form's way in, for few rows (bf16 weights, R a multiple of 8): q fp32 [n][H][dn + dr] -> qa[h][t][r] = sum_d uk[h][d][r]
+ * * q[t][h][d] and qr[t][h][dr] as ao_lm_latent_query_prep makes it; both fp32. */
+AO_B200_API int ao_lm_latent_query_fold(const float* q, const void* uk, int dt, int64_t n, int H, int dn, int dr, int R, int rot_dims,
+                                        const float* inv_freq, float amp, const int32_t* pos, float* qa, float* qr, void* stream);
 /* The folded form's way back, for few rows: out[t][h * dv + j] = sigmoid(gate[t][h * dv + j]) * sum_r uv[h][j][r] * olat[t][h][r]
  * (olat, uv, out in `dt`; gate fp32 logits with row stride ld_gate, null: none).  ao_lm_sigmoid_gate_rows: y *= sigmoid(gate). */
 AO_B200_API int ao_lm_latent_value_up(const void* olat, const void* uv, int dt, int64_t n, int H, int R, int dv, const float* gate,
                                       int64_t ld_gate, void* out, int64_t ld_out, void* stream);
 AO_B200_API int ao_lm_sigmoid_gate_rows(const float* gate, int64_t ld_gate, int64_t n, int64_t cols, void* y, int64_t ld, int dt,
                                         void* stream);
+
+/* Products of up to 8 rows with a bf16 weight matrix: out[t][m] = sum_k w[m][k] x[t][k], row strides ld_x, ld_w, ld_out; K, ld_x and
+ * ld_w multiples of 8, x and w on 16-byte boundaries (else AO_B200_ERR_UNSUPPORTED).  act 0: fp32 result; 1: its squared ReLU in
+ * bf16.  The weights (here, of ao_lm_latent_query_fold and of ao_lm_latent_value_up) may be read before the launch in front has
+ * finished: they must not be written by a launch in flight. */
+AO_B200_API int ao_lm_gemv_rows(const void* x, int64_t ld_x, const void* w, int64_t ld_w, int64_t n, int64_t M, int64_t K, int act, void* out,
+                                int64_t ld_out, void* stream);
 
 #ifdef __cplusplus
 }

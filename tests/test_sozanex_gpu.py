@@ -262,6 +262,51 @@ def test_value_up_projection_with_the_gate(dtype, n, H, R, dv):
     assert float((out[:, H * dv:].float() - 9).abs().max()) == 0.0
 
 
+@pytest.mark.parametrize("n", [1, 2, 3, 8])
+@pytest.mark.parametrize("M,K,pad", [(37, 96, 0), (2048, 2048, 8), (5, 8, 16), (1000, 9216, 0), (4608, 264, 8), (3, 20000, 0)])
+def test_products_of_few_rows(n, M, K, pad):
+    lib, L = _lm()
+    g = _gen(M)
+    x, w = torch.randn(n, K + pad, generator=g).bfloat16(), (torch.randn(M, K + pad, generator=g) / math.sqrt(K)).bfloat16()
+    xd, wd = x.cuda(), w.cuda()
+    torch.cuda.synchronize()
+    ref = x[:, :K].double() @ w[:, :K].double().T
+    out, ya = torch.full((n, M + 3), 9.0, device="cuda"), torch.full((n, M + 3), 9.0, device="cuda", dtype=torch.bfloat16)
+    for o, act in ((out, 0), (ya, 1)):
+        lib.lm_check(L.ao_lm_gemv_rows(_p(xd), K + pad, _p(wd), K + pad, n, M, K, act, _p(o), M + 3, _st()), "gemv")
+        assert _close(o[:, :M].float(), O.squared_relu(ref) if act else ref, 1e-2 if act else 2e-5)
+        assert float((o[:, M:].float() - 9).abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("n,H,dn,dr,dims,R", [(1, 3, 8, 4, 4, 16), (8, 2, 200, 6, 2, 96), (2, 16, 128, 64, 64, 512), (3, 1, 1, 2, 0, 8)])
+def test_query_fold_of_few_rows(n, H, dn, dr, dims, R):
+    lib, L = _lm()
+    g = _gen(R + dn)
+    q, uk = torch.randn(n, H, dn + dr, generator=g), (torch.randn(H, dn, R, generator=g) / math.sqrt(dn)).bfloat16()
+    pos = [5, 0, 999, 17, 3, 8, 1, 2][:n]
+    rot = O.rotary(dims, 300.0, ramp=(4.0, 64, 8.0, 1.0)) if dims else None
+    f, amp = O.frequencies(rot) if dims else (torch.ones(1), 1.0)
+    qd, ukd, fd, pd = q.cuda(), uk.cuda(), f.float().cuda(), _i32(pos)
+    torch.cuda.synchronize()
+    qa, qr = torch.zeros(H, n, R, device="cuda"), torch.zeros(n, H, dr, device="cuda")
+    lib.lm_check(L.ao_lm_latent_query_fold(_p(qd), _p(ukd), BF16, n, H, dn, dr, R, dims, _p(fd), amp, _p(pd), _p(qa), _p(qr), _st()), "query_fold")
+    assert _close(qa, torch.einsum("thd,hdr->htr", q[..., :dn].double(), uk.double()))
+    assert _close(qr, O.rotate(q[..., dn:].double(), torch.tensor(pos), rot, "interleaved"), 1e-4)
+
+
+@pytest.mark.parametrize("V,ld", [(1, 1), (7, 8), (4096, 4096), (32000, 32001), (128256, 128256)])
+def test_greedy_choice_takes_the_first_of_equals(V, ld):
+    lib, L = _lm()
+    z = torch.randn(3, ld, generator=_gen(V))
+    hot = [V - 1, V // 2, min(V - 1, 5)]
+    for b, i in enumerate(hot):
+        z[b, i] = 50.0
+    z[1, -1 if ld == V else V:] = 50.0                      # a later equal one (or one past the vocabulary)
+    zd, out = z.cuda(), torch.zeros(3, dtype=torch.int64, device="cuda")
+    lib.lm_check(L.ao_lm_argmax(_p(zd), ld, 3, V, _p(out), _st()), "argmax")
+    assert out.tolist() == hot
+
+
 @pytest.mark.parametrize("types", [(F32, F32), (F32, BF16), (BF16, BF16)])
 @pytest.mark.parametrize("n,cols", [(3, 37), (2, 4096), (300, 64), (1, 20000)])
 def test_squared_relu_rows(types, n, cols):

@@ -234,6 +234,8 @@ LM_SIGNATURES = {
                                     _vp, _vp, _vp, _vp, _vp, _vp],
     "ao_lm_gated_latent_attention_expanded": [_vp, _vp, _vp, _i64, _vp, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i64, _i32, _i32, _i32,
                                               _i32, _f32, _i32, _vp, _vp, _i64, _vp, _i64, _vp],
+    "ao_lm_latent_query_fold": [_vp, _vp, _i32, _i64, _i32, _i32, _i32, _i32, _i32, _vp, _f32, _vp, _vp, _vp, _vp],
+    "ao_lm_gemv_rows": [_vp, _i64, _vp, _i64, _i64, _i64, _i64, _i32, _vp, _i64, _vp],
     "ao_lm_latent_value_up": [_vp, _vp, _i32, _i64, _i32, _i32, _i32, _vp, _i64, _vp, _i64, _vp],
     "ao_lm_sigmoid_gate_rows": [_vp, _i64, _i64, _i64, _vp, _i64, _i32, _vp],
 }

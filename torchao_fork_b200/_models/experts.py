@@ -9,6 +9,7 @@ from typing import Optional
 import torch
 
 from .. import _lib
+from .products import ACT_SQUARED_RELU, gemv, gemv_takes, mm_f32
 
 
 def _p(t: Optional[torch.Tensor]):
@@ -21,8 +22,8 @@ def glu_unit(L, dt, x: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, l
     gu = torch.mm(x, w_gu.t())
     ya = torch.empty(n, ff, dtype=x.dtype, device=x.device)
     _lib.lm_check(L.ao_lm_glu_act_shift(_p(gu), dt, n, ff, limit, alpha, shift, _p(ya), st), "glu_act")
-    if f32_out and x.dtype == torch.bfloat16:
-        return torch.mm(ya, w_down.t(), out_dtype=torch.float32), 3
+    if f32_out:
+        return mm_f32(L, ya, w_down), 3
     return torch.mm(ya, w_down.t()), 3
 
 
@@ -33,11 +34,14 @@ def act_unit(L, dt, x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, r
     """One ungated unit over all rows: GEMM up -> squared ReLU (times row_scale[t], fp32 [n], when given) -> GEMM down.
     -> ([n][W], launches)."""
     n, ff = x.shape[0], w_down.shape[1]
+    if row_scale is None and gemv_takes(x, w_up):       # few rows: the activation joins the first product
+        ya = gemv(L, x, w_up, ACT_SQUARED_RELU)
+        return (mm_f32(L, ya, w_down), 2) if f32_out else (torch.mm(ya, w_down.t()), 2)
     u = torch.mm(x, w_up.t())
     ya = torch.empty(n, ff, dtype=x.dtype, device=x.device)
     _lib.lm_check(L.ao_lm_unary_rows(_p(u), dt, n, ff, ACT_RELU2, 0.0, _p(row_scale), 1, _p(ya), dt, st), "unary_rows")
-    if f32_out and x.dtype == torch.bfloat16:
-        return torch.mm(ya, w_down.t(), out_dtype=torch.float32), 3
+    if f32_out:
+        return mm_f32(L, ya, w_down), 3
     return torch.mm(ya, w_down.t()), 3
 
 

@@ -251,11 +251,8 @@ class StepEngine(SegmentStepEngine):
         xn = torch.empty(k, cfg.width, dtype=m.dtype, device=dev)
         _lib.lm_check(self.L.ao_lm_add_layer_norm(_p(x), None, 0.0, _p(d_rows), k, cfg.width, _p(m.final_norm), _p(m.final_norm_b),
                                                   self.dt, cfg.norm_eps, None, _p(xn), st), "add_layer_norm")
-        lg = self._mm_f32(xn, m.head)
+        lg = self._mm_f32(xn, m.head, out)
         if cfg.logit_softcap:
             _lib.lm_check(self.L.ao_lm_unary_rows(_p(lg), _lib.DT_F32, k, cfg.vocab_size, ACT_SOFTCAP, cfg.logit_softcap, None, 0,
                                                   _p(lg), _lib.DT_F32, st), "unary_rows")
-        if out is not None:
-            out.copy_(lg)
-            return out
         return lg

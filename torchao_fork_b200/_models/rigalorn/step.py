@@ -129,8 +129,9 @@ class StepEngine(SoftmaxStepEngine):
         rot = (a.rot.dims, _p(lay.inv_freq), a.rot.amplitude)
         _lib.lm_check(L.ao_lm_latent_low_prep(_p(proj), lay.ld, n, lay.q_off, Rq, lay.kv_off, R, dr, _p(lay.q_norm), _p(lay.c_norm), dt,
                                               self.cfg.norm_eps, *rot, _p(meta.pos), _p(cq), _p(c), _p(kr), st), "latent_low_prep")
-        qn, qr = self._latent_queries(lay, a, cq, meta, st)
-        launches = 4 + self._latent_attend(lay, a, self._shape(la, ls), cache, c, kr, qn, qr, row, meta, st)
+        shape = self._shape(la, ls)
+        q, qr, k = self._latent_queries(lay, a, shape, cq, meta, st)
+        launches = 2 + k + self._latent_attend(lay, a, shape, cache, c, kr, q, qr, row, meta, st)
         _lib.lm_check(L.ao_lm_ring_append(_p(c), _p(kr), n, R, dr, cache.c.shape[1], dt, _p(meta.slot), _p(meta.pos), _p(meta.ahead),
                                           _p(cache.c), _p(cache.kr), st), "ring_append")
         return launches
@@ -141,8 +142,4 @@ class StepEngine(SoftmaxStepEngine):
         xn = torch.empty(k, cfg.width, dtype=m.dtype, device=self.dev)
         _lib.lm_check(self.L.ao_lm_add_rms_norm(_p(x), None, _p(d_rows), k, cfg.width, _p(m.final_norm), self.dt, cfg.norm_eps, _p(xn), st),
                       "add_rms_norm")
-        lg = self._mm_f32(xn, m.head)
-        if out is not None:
-            out.copy_(lg)
-            return out
-        return lg
+        return self._mm_f32(xn, m.head, out)

@@ -13,6 +13,7 @@ import numpy as np
 import torch
 
 from .. import _lib
+from .products import mm_f32
 
 # a portion longer than this is cut into pieces (bounds the workspace)
 MAX_STEP_TOKENS = 4096
@@ -42,6 +43,7 @@ class StepMeta:
     attn: Dict[tuple, tuple]   # attention shape -> (tile_first, tile_count, n_tiles, tensor-core form?)
     seg: tuple           # (first row, rows, n) of the step's segments, whole
     rec: Optional[tuple] = None   # tiles of the matrix-state recurrences (as `scan`), when some segment is longer than one tile
+    all_rows: bool = False        # the logits of every row are wanted, in order (a decode step)
     extra: Dict[tuple, torch.Tensor] = {}   # a family's own int32 tables (`_piece_tables`)
 
 
@@ -231,11 +233,9 @@ class SegmentStepEngine:
         d_tok, meta = self._meta(slot, pos, tok)
         return self._layers(d_tok, meta)
 
-    def _mm_f32(self, a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    def _mm_f32(self, a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """a @ w^T with an fp32 result (what fp32 kernels read next)."""
-        if a.dtype == torch.bfloat16:
-            return torch.mm(a, w.t(), out_dtype=torch.float32)
-        return torch.mm(a, w.t())
+        return mm_f32(self.L, a, w, out)
 
     def _splits(self, ctas: int, chunk: int) -> int:
         """Key splits of the fp32 attention kernel: enough CTAs to fill the GPU when few rows attend over a long chunk
@@ -297,6 +297,7 @@ class GraphDecodeEngine:
         meta.scan = (ar, ones, B, None, None, 0)       # one row per sequence: every tile is a whole segment
         meta.attn = {shape: (ar, ones, B, False) for shape in self.eng.attn_keys}
         meta.seg = (ar, ones, B)
+        meta.all_rows = True
         self.meta, self.pos, self.rows = meta, meta.pos, ar
         self.graph = None
         self.graph_stream = None

@@ -10,6 +10,7 @@ import numpy as np
 import torch
 
 from .. import _lib
+from .products import GEMV_ROWS
 from .segment_step import SegmentStepEngine, StepMeta, _p
 
 PAIR_INTERLEAVED, PAIR_HALVES = 0, 1      # rotation couples (2i, 2i + 1) / (i, i + dims / 2)
@@ -103,18 +104,25 @@ class SoftmaxStepEngine(SegmentStepEngine):
                                                  _p(meta.slot), _p(meta.pos), _p(meta.ahead), _p(cache.k), _p(cache.v), _p(cache.k_first),
                                                  _p(cache.v_first), st), "window_append")
 
-    def _latent_queries(self, lay, a, cq, meta: StepMeta, st):
-        """Up-projected queries -> unrotated parts head-major in the storage type, rotated parts in fp32 (2 launches)."""
-        H, dn, dr, n = a.heads, a.dim, a.rot_dim, meta.n
+    def _latent_queries(self, lay, a, shape, cq, meta: StepMeta, st):
+        """Up-projected queries, split: -> (unrotated parts, rotated parts fp32 [n][H][dr], launches).  Unrotated parts: head-major in
+        the storage type for the expanded form, multiplied by the key up-projection (fp32 [H][n][R]) for the folded one."""
+        H, dn, dr, R, n = a.heads, a.dim, a.rot_dim, a.kv_rank, meta.n
         q = self._mm_f32(cq, lay.uq)
-        qn, qr = torch.empty(H, n, dn, dtype=self.m.dtype, device=self.dev), torch.empty(n, H, dr, dtype=torch.float32, device=self.dev)
-        _lib.lm_check(self.L.ao_lm_latent_query_prep(_p(q), n, H, dn, dr, self.dt, a.rot.dims, _p(lay.inv_freq), a.rot.amplitude,
-                                                     _p(meta.pos), _p(qn), _p(qr), st), "latent_query_prep")
-        return qn, qr
+        qr = torch.empty(n, H, dr, dtype=torch.float32, device=self.dev)
+        rot = (a.rot.dims, _p(lay.inv_freq), a.rot.amplitude, _p(meta.pos))
+        folded = not meta.attn[shape][3]
+        if folded and n <= GEMV_ROWS and self.m.dtype == torch.bfloat16 and R % 8 == 0:
+            qa = torch.empty(H, n, R, dtype=torch.float32, device=self.dev)
+            _lib.lm_check(self.L.ao_lm_latent_query_fold(_p(q), _p(lay.uk), self.dt, n, H, dn, dr, R, *rot, _p(qa), _p(qr), st), "latent_query_fold")
+            return qa, qr, 2
+        qn = torch.empty(H, n, dn, dtype=self.m.dtype, device=self.dev)
+        _lib.lm_check(self.L.ao_lm_latent_query_prep(_p(q), n, H, dn, dr, self.dt, *rot, _p(qn), _p(qr), st), "latent_query_prep")
+        return (self._bmm_f32(qn, lay.uk), qr, 3) if folded else (qn, qr, 2)
 
-    def _latent_attend(self, lay, a, shape, cache, c, kr, qn, qr, row, meta: StepMeta, st, sink=None, gate=None):
-        """Softmax of the step's queries over the cached latents and the step's own, into the first columns of `row` ->
-        launches.  sink: a logit per head in every denominator; gate: (address, row stride) of fp32 logits per output column.
+    def _latent_attend(self, lay, a, shape, cache, c, kr, q, qr, row, meta: StepMeta, st, sink=None, gate=None):
+        """Softmax of the step's queries (as `_latent_queries` left them) over the cached latents and the step's own, into the first
+        columns of `row` -> launches.  sink: a logit per head in every denominator; gate: (address, row stride) of fp32 logits per output column.
         Prompt portions attend over up-projected keys and values, few rows over the latents themselves."""
         L, dt, dev, tdt = self.L, self.dt, self.dev, self.m.dtype
         H, dn, dr, dv, R, n = a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, meta.n
@@ -131,18 +139,17 @@ class SoftmaxStepEngine(SegmentStepEngine):
             kv = torch.mm(c, lay.ukv.t())                                              # [rows][H dn | H dv]
             ld = H * (dn + dv)
             _lib.lm_check(L.ao_lm_gated_latent_attention_expanded(
-                _p(qn), _p(qr), _p(kv), ld, kv.data_ptr() + kv.element_size() * H * dn, ld, _p(kr), dt, _p(meta.pos), _p(tf), _p(tc),
+                _p(q), _p(qr), _p(kv), ld, kv.data_ptr() + kv.element_size() * H * dn, ld, _p(kr), dt, _p(meta.pos), _p(tf), _p(tc),
                 _p(meta.extra[("key0", window)]), nt, n, H, dn, dr, dv, a.scale, window, _p(sink), g_ptr, g_ld, _p(row), row.shape[1], st),
                 "gated_latent_attention_expanded")
             return launches
-        qa = self._bmm_f32(qn, lay.uk)                                                 # fp32 [H][n][R]
         ns = self._splits(nt * -(-H // 16), window)
         ws = torch.empty(max(16, int(L.ao_lm_latent_attention_workspace_bytes(n, H, R, ns))), dtype=torch.uint8, device=dev)
         olat = torch.empty(n, H, R, dtype=tdt, device=dev)
-        _lib.lm_check(L.ao_lm_window_latent_attention(_p(qa), _p(qr), _p(cache.c), _p(cache.kr), _p(c), _p(kr), dt, ring, _p(meta.slot),
+        _lib.lm_check(L.ao_lm_window_latent_attention(_p(q), _p(qr), _p(cache.c), _p(cache.kr), _p(c), _p(kr), dt, ring, _p(meta.slot),
                                                       _p(meta.pos), _p(meta.back), _p(tf), _p(tc), nt, n, H, R, dr, a.scale, window,
                                                       _p(sink), None, ns, _p(ws), ws.numel(), _p(olat), st), "window_latent_attention")
-        launches = 3 if ns > 1 else 2
+        launches = 2 if ns > 1 else 1
         if n <= VALUE_UP_ROWS:
             _lib.lm_check(L.ao_lm_latent_value_up(_p(olat), _p(lay.uv), dt, n, H, R, dv, g_ptr, g_ld, _p(row), row.shape[1], st),
                           "latent_value_up")

@@ -16,11 +16,12 @@ registers.
       part, the cache's new rows) -> GEMM W_uq -> `latent_query_prep` -> then
       for prompt portions: the visible latents made contiguous, ONE GEMM for all heads' keys and values,
           `gated_latent_attention_expanded` (sink in the denominator, sigmoid gate on the way out);
-      for few rows: batched GEMM that folds the key up-projection into the queries, `window_latent_attention` over the latents
-          themselves (sink), `latent_value_up` (value up-projection and sigmoid gate);
+      for few rows: `latent_query_fold` instead (the key up-projection folded into the queries), `window_latent_attention` over the
+          latents themselves (sink), `latent_value_up` (value up-projection and sigmoid gate);
       -> GEMM W_o.
-  feed-forward: GEMM up -> squared ReLU -> GEMM down; for few rows both products are matrix-vector kernels, the first with the
-      activation in it.
+  feed-forward: GEMM up -> squared ReLU -> GEMM down.
+For up to eight rows in bf16 every product is `gemv_rows`, whose weights travel while the kernel in front finishes; the one in front
+of the squared ReLU has it built in.
 Norms, rotations, attention scores and weights, and the residual are fp32 in both storage types.
 
 `StepEngine.step` is what prefill, the trace runner and tests call; `GraphDecodeEngine` wraps the same layer loop for
@@ -38,6 +39,7 @@ from .model import Sozanex
 class StepEngine(SoftmaxStepEngine):
     def __init__(self, model: Sozanex):
         super().__init__(model)
+        self._normed = None     # a decode step's rows behind the output norm
         self.plan = [(r, i, begins) for r, (i, begins) in enumerate(self.cfg.schedule)]
 
     def _layer_runs(self):
@@ -99,6 +101,8 @@ class StepEngine(SoftmaxStepEngine):
                 launches += 1
                 if nxt is None:
                     break
+            if nxt is None and meta.all_rows:       # every row's logits are wanted: the closing kernel takes the output norm as well
+                nxt = m.final_norm
             if begins:
                 h = self._close(x, y, post_w, y_bias, None, st, cast=True)
                 h = self._close(x, self._mm_f32(h, m.loop_in[:W]), None, None, nxt, st, add=y0)
@@ -106,6 +110,7 @@ class StepEngine(SoftmaxStepEngine):
             else:
                 h = self._close(x, y, post_w, y_bias, nxt, st)
             launches += 1
+        self._normed = h if meta.all_rows and after_run is None else None
         self.launches = launches
         return x
 
@@ -138,9 +143,9 @@ class StepEngine(SoftmaxStepEngine):
                                                     self.cfg.norm_eps, a.rot.dims, _p(lay.inv_freq), a.rot.amplitude, _p(meta.pos),
                                                     _p(meta.slot), cache.c.shape[1], _p(cq), _p(c), _p(kr), _p(cache.c) if full else None,
                                                     _p(cache.kr) if full else None, st), "latent_low_prep_store")
-        qn, qr = self._latent_queries(lay, a, cq, meta, st)
-        launches = 3 + self._latent_attend(lay, a, self._shape(la, rs), cache, c, kr, qn, qr, o, meta, st, lay.sink,
-                                           (proj.data_ptr() + 4 * lay.g_off, lay.ld))
+        shape = self._shape(la, rs)
+        q, qr, k = self._latent_queries(lay, a, shape, cq, meta, st)
+        launches = 1 + k + self._latent_attend(lay, a, shape, cache, c, kr, q, qr, o, meta, st, lay.sink, (proj.data_ptr() + 4 * lay.g_off, lay.ld))
         if not full:
             _lib.lm_check(L.ao_lm_ring_append(_p(c), _p(kr), n, R, dr, cache.c.shape[1], dt, _p(meta.slot), _p(meta.pos), _p(meta.ahead),
                                               _p(cache.c), _p(cache.kr), st), "ring_append")
@@ -150,11 +155,9 @@ class StepEngine(SoftmaxStepEngine):
     def _logits_dev(self, x, d_rows, k, out=None):
         m, cfg = self.m, self.cfg
         st = torch.cuda.current_stream(self.dev).cuda_stream
-        xn = torch.empty(k, cfg.width, dtype=m.dtype, device=self.dev)
-        _lib.lm_check(self.L.ao_lm_add_layer_norm(_p(x), None, 0.0, _p(d_rows), k, cfg.width, _p(m.final_norm), None, self.dt, cfg.norm_eps,
-                                                  None, _p(xn), st), "add_layer_norm")
-        lg = self._mm_f32(xn, m.head)
-        if out is not None:
-            out.copy_(lg)
-            return out
-        return lg
+        xn, self._normed = self._normed, None
+        if xn is None:
+            xn = torch.empty(k, cfg.width, dtype=m.dtype, device=self.dev)
+            _lib.lm_check(self.L.ao_lm_add_layer_norm(_p(x), None, 0.0, _p(d_rows), k, cfg.width, _p(m.final_norm), None, self.dt, cfg.norm_eps,
+                                                      None, _p(xn), st), "add_layer_norm")
+        return self._mm_f32(xn, m.head, out)

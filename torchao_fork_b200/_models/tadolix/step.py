@@ -159,8 +159,4 @@ class StepEngine(SegmentStepEngine):
         xn = torch.empty(k, cfg.width, dtype=m.dtype, device=dev)
         _lib.lm_check(self.L.ao_lm_streams_norm(_p(x), _p(d_rows), k, max(1, cfg.streams), cfg.width, None, _p(m.final_norm),
                                                 self.dt, 1.0, cfg.norm_eps, None, _p(xn), st), "streams_norm")
-        lg = self._mm_f32(xn, m.head)
-        if out is not None:
-            out.copy_(lg)
-            return out
-        return lg
+        return self._mm_f32(xn, m.head, out)

@@ -129,6 +129,8 @@ latent_attn_kernel(const float* __restrict__ qa, const float* __restrict__ qr, c
                    int tiles_per_split, int n_split, const T* __restrict__ sink, const float* __restrict__ gate,
                    T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, WindowArgs<T> win) {
   extern __shared__ float smem[];
+  pdl_trigger();
+  pdl_wait();
   const int D = R + dr, DP = D + 1;
   float* qs = smem;                         // [kWarps][D][4]
   float* ks = smem + (size_t)kWarps * D * 4;  // [kKeys][DP]
@@ -339,6 +341,8 @@ latent_attn_mma_kernel(const float* __restrict__ qa, const float* __restrict__ q
   using T = __nv_bfloat16;
   constexpr int R = 64 * NT;
   extern __shared__ float smem[];
+  pdl_trigger();
+  pdl_wait();
   const int D = R + dr, DP = D + 4;            // pitch = 4 or 20 mod 32: fragment loads along rows hit 32 banks
   float* qhi = smem;                           // [16][DP]
   float* qlo = qhi + kMmaRows * DP;            // [16][DP]
@@ -528,44 +532,77 @@ __host__ __device__ inline bool mma_path(int dt, int H, int R, int dr) {
   return dt == AO_LM_BF16 && R % 64 == 0 && R <= 512 && dr % 16 == 0;
 }
 
-// one CTA per (token, head): merges the key splits that hold keys this token sees, then sink, gate, normalisation
-template <typename T>
-__global__ void latent_attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                         const int32_t* __restrict__ pos, int H, int R, int tiles_per_split, int n_split,
-                                         const T* __restrict__ sink, const float* __restrict__ gate, T* __restrict__ out,
-                                         int window) {
-  __shared__ float wsplit[64];   // n_split <= 64: exp(m_s - top) / denominator, gate folded in
+// One CTA per (token, head) and 128 output coordinates: merges the key splits that hold keys this token sees, then sink, gate,
+// normalisation.  A warp takes every kMergeWarps-th split, all its loads in flight at once (four coordinates per lane).
+constexpr int kMergeWarps = 8;
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kMergeWarps * 32)
+latent_attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int32_t* __restrict__ pos, int H, int R,
+                         int tiles_per_split, int n_split, const T* __restrict__ sink, const float* __restrict__ gate, T* __restrict__ out,
+                         int window) {
+  constexpr int kPer = 64 / kMergeWarps;      // n_split <= 64
+  __shared__ __align__(16) float sums[kMergeWarps][128];
+  pdl_trigger();
+  pdl_wait();
   const int64_t row = blockIdx.x;
   const int64_t t = row / H;
-  const int h = (int)(row - t * H);
+  const int h = (int)(row - t * H), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // the splits that may hold keys of this row (under a window every split left its statistics)
   const int ns = window != kNoWindow ? n_split : min(n_split, pos[t] / (tiles_per_split * kKeys) + 1);
-  if (threadIdx.x < 32) {
-    const int lane = threadIdx.x;
-    const float sk = sink ? ldf(sink + h) : -INFINITY;
-    float m_a = lane < ns ? part_ml[(row * n_split + lane) * 2] : -INFINITY;
-    float m_b = lane + 32 < ns ? part_ml[(row * n_split + lane + 32) * 2] : -INFINITY;
-    const float top = fmaxf(warp_max(fmaxf(m_a, m_b)), sk);
-    const float e_a = lane < ns ? __expf(m_a - top) : 0.f, e_b = lane + 32 < ns ? __expf(m_b - top) : 0.f;
-    float den = (lane < ns ? part_ml[(row * n_split + lane) * 2 + 1] * e_a : 0.f) +
-                (lane + 32 < ns ? part_ml[(row * n_split + lane + 32) * 2 + 1] * e_b : 0.f);
-    den = warp_sum(den) + __expf(sk - top);
-    const float k = (gate ? gate[row] : 1.f) / den;
-    wsplit[lane] = e_a * k;
-    wsplit[lane + 32] = e_b * k;
+  const float2* ml = reinterpret_cast<const float2*>(part_ml) + row * n_split;
+  const float2 a = lane < ns ? ml[lane] : make_float2(-INFINITY, 0.f), b = lane + 32 < ns ? ml[lane + 32] : make_float2(-INFINITY, 0.f);
+  const float sk = sink ? ldf(sink + h) : -INFINITY;
+  const float top = fmaxf(warp_max(fmaxf(a.x, b.x)), sk);
+  const float e_a = __expf(a.x - top), e_b = __expf(b.x - top);
+  const float den = warp_sum(a.y * e_a + b.y * e_b) + __expf(sk - top);
+  const float k = (gate ? gate[row] : 1.f) / den;
+  // weight of split warp + i * kMergeWarps; 0: a split that saw no key may have left no sums
+  float w[kPer];
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
+    const int s = warp + i * kMergeWarps;
+    w[i] = __shfl_sync(0xffffffffu, s < 32 ? e_a : e_b, s & 31) * k;
+    if (s >= ns) w[i] = 0.f;
   }
-  __syncthreads();
-  // blockIdx.y: which 128 output coordinates (one per thread), so that a decoded token's few rows still fill many SMs
-  const int d = blockIdx.y * blockDim.x + threadIdx.x;
-  if (d < R) {
-    float acc = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < ns; ++s) {
-      const float w = wsplit[s];     // 0: a split that saw no key may have left no sums
-      acc = w != 0.f ? fmaf(part_o[(row * n_split + s) * R + d], w, acc) : acc;
+  const int d0 = blockIdx.y * 128 + lane * 4;
+  float4 v[kPer];
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
+    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float* p = part_o + (row * n_split + warp + i * kMergeWarps) * (int64_t)R + d0;
+    if (w[i] != 0.f) {
+      if (VEC) {
+        if (d0 < R) v[i] = ld4(p);
+      } else {
+        if (d0 < R) v[i].x = p[0];
+        if (d0 + 1 < R) v[i].y = p[1];
+        if (d0 + 2 < R) v[i].z = p[2];
+        if (d0 + 3 < R) v[i].w = p[3];
+      }
     }
-    stf(out + row * R + d, acc);
   }
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < kPer; ++i)
+    acc.x = fmaf(v[i].x, w[i], acc.x), acc.y = fmaf(v[i].y, w[i], acc.y), acc.z = fmaf(v[i].z, w[i], acc.z), acc.w = fmaf(v[i].w, w[i], acc.w);
+  *reinterpret_cast<float4*>(&sums[warp][lane * 4]) = acc;
+  __syncthreads();
+  const int d = blockIdx.y * 128 + threadIdx.x;
+  if (threadIdx.x < 128 && d < R) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMergeWarps; ++i) s += sums[i][threadIdx.x];
+    stf(out + row * R + d, s);
+  }
+}
+
+template <typename T>
+int launch_merge(int64_t n, int H, int R, int tps, int n_split, const float* part_o, const float* part_ml, const int32_t* pos, const void* sink,
+                 const float* gate, void* out, int window, cudaStream_t st) {
+  const bool vec = R % 4 == 0 && reinterpret_cast<uintptr_t>(part_o) % 16 == 0;
+  auto kern = vec ? latent_attn_merge_kernel<T, true> : latent_attn_merge_kernel<T, false>;
+  return lm_launch_early(kern, dim3((unsigned)(n * H), (unsigned)((R + 127) / 128)), dim3(kMergeWarps * 32), 0, st, part_o, part_ml, pos, H, R, tps,
+                         n_split, static_cast<const T*>(sink), gate, static_cast<T*>(out), window);
 }
 
 // 32-key tiles that a row tile of `tile_tokens` tokens can see: keys 0 .. max_pos, or a window's worth of them
@@ -596,13 +633,11 @@ int launch(const float* qa, const float* qr, const void* c_cache, const void* kr
   const int tps = (tiles + n_split - 1) / n_split;
   const int quads = (H + 3) / 4;
   dim3 grid((unsigned)n_tiles, (unsigned)((quads + HQ - 1) / HQ), (unsigned)n_split);
-  kern<<<grid, kWarps * 32, smem, st>>>(qa, qr, static_cast<const T*>(c_cache), static_cast<const T*>(kr_cache), S, slot, pos,
-                                        tile_first, tile_count, n, H, R, dr, scale, HQ, tps, n_split,
-                                        static_cast<const T*>(sink), gate, static_cast<T*>(out), part_o, part_ml, win);
-  if (n_split > 1)
-    latent_attn_merge_kernel<T><<<dim3((unsigned)(n * H), (unsigned)((R + 127) / 128)), 128, 0, st>>>(part_o, part_ml, pos, H, R, tps, n_split,
-                                                                  static_cast<const T*>(sink), gate, static_cast<T*>(out), win.window);
-  return lm_launch_status();
+  const int rc = lm_launch_early(kern, grid, dim3(kWarps * 32), smem, st, qa, qr, static_cast<const T*>(c_cache), static_cast<const T*>(kr_cache),
+                                 S, slot, pos, tile_first, tile_count, n, H, R, dr, scale, HQ, tps, n_split, static_cast<const T*>(sink), gate,
+                                 static_cast<T*>(out), part_o, part_ml, win);
+  if (rc != AO_B200_OK || n_split == 1) return rc;
+  return launch_merge<T>(n, H, R, tps, n_split, part_o, part_ml, pos, sink, gate, out, win.window, st);
 }
 
 template <int NT>
@@ -627,13 +662,11 @@ int launch_mma(const float* qa, const float* qr, const void* c_cache, const void
   const int tiles = key_tiles(max_pos, win.window, kMmaRows / HB);
   const int tps = (tiles + n_split - 1) / n_split;
   dim3 grid((unsigned)n_tiles, (unsigned)((H + HB - 1) / HB), (unsigned)n_split);
-  kern<<<grid, kWarps * 32, smem, st>>>(qa, qr, static_cast<const T*>(c_cache), static_cast<const T*>(kr_cache), S, slot, pos,
-                                        tile_first, tile_count, n, H, dr, scale, HB, tps, n_split, static_cast<const T*>(sink),
-                                        gate, static_cast<T*>(out), part_o, part_ml, win);
-  if (n_split > 1)
-    latent_attn_merge_kernel<T><<<dim3((unsigned)(n * H), (unsigned)((R + 127) / 128)), 128, 0, st>>>(part_o, part_ml, pos, H, R, tps, n_split,
-                                                                  static_cast<const T*>(sink), gate, static_cast<T*>(out), win.window);
-  return lm_launch_status();
+  const int rc = lm_launch_early(kern, grid, dim3(kWarps * 32), smem, st, qa, qr, static_cast<const T*>(c_cache), static_cast<const T*>(kr_cache),
+                                 S, slot, pos, tile_first, tile_count, n, H, dr, scale, HB, tps, n_split, static_cast<const T*>(sink), gate,
+                                 static_cast<T*>(out), part_o, part_ml, win);
+  if (rc != AO_B200_OK || n_split == 1) return rc;
+  return launch_merge<T>(n, H, R, tps, n_split, part_o, part_ml, pos, sink, gate, out, win.window, st);
 }
 
 }  // namespace
@@ -646,7 +679,7 @@ extern "C" int ao_lm_latent_attention_plan(int dt, int H, int R, int dr, int* ti
 
 extern "C" int64_t ao_lm_latent_attention_workspace_bytes(int64_t n, int H, int R, int n_split) {
   if (n_split <= 1) return 0;
-  return n * H * n_split * (int64_t)(R + 2) * 4;
+  return n * H * n_split * (int64_t)(R + 2) * 4 + 16;
 }
 
 template <typename T>
@@ -659,8 +692,8 @@ static int dispatch_latent(const float* qa, const float* qr, const void* c_cache
   float *part_o = nullptr, *part_ml = nullptr;
   if (n_split > 1) {
     if (!workspace || workspace_bytes < ao_lm_latent_attention_workspace_bytes(n, H, R, n_split)) return AO_B200_ERR_WORKSPACE;
-    part_o = static_cast<float*>(workspace);
-    part_ml = part_o + n * H * n_split * (int64_t)R;
+    part_ml = static_cast<float*>(workspace);                                  // pairs, then sums on a 16-byte boundary
+    part_o = part_ml + (n * H * n_split * (int64_t)2 + 3) / 4 * 4;
   }
 #define LM_ARGS qa, qr, c_cache, kr_cache, S, slot, pos, tile_first, tile_count, n_tiles, n, H
 #define LM_TAIL dr, scale, sink, gate, max_pos, n_split, part_o, part_ml, out, win, st

@@ -36,7 +36,29 @@ static inline int lm_launch_status() {
 }
 static inline cudaStream_t lm_stream(void* s) { return static_cast<cudaStream_t>(s); }
 
+// Launch that may start while the kernel in front of it still runs (programmatic dependent launch).  The kernel calls
+// lm::pdl_wait() in EVERY thread before it touches anything that an earlier launch writes or still reads, and before any return;
+// until then it may read weights.  A kernel in front that calls lm::pdl_trigger() lets it start early; without that it starts
+// when the one in front ends.
+template <typename... P, typename... A>
+static inline int lm_launch_early(void (*kern)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, A... args) {
+  cudaLaunchConfig_t c = {};
+  c.gridDim = grid, c.blockDim = block, c.dynamicSmemBytes = smem, c.stream = st;
+  cudaLaunchAttribute at[1];
+  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  at[0].val.programmaticStreamSerializationAllowed = 1;
+  c.attrs = at, c.numAttrs = 1;
+  const cudaError_t e = cudaLaunchKernelEx(&c, kern, static_cast<P>(args)...);
+  if (e == cudaSuccess) return AO_B200_OK;
+  (void)cudaGetLastError();
+  g_lm_last_cuda_error = (int)e;
+  return AO_B200_ERR_CUDA;
+}
+
 namespace lm {
+
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
 __device__ __forceinline__ float ldf(const float* p) { return *p; }
 __device__ __forceinline__ float ldf(const __nv_bfloat16* p) { return __bfloat162float(*p); }

@@ -112,6 +112,8 @@ __global__ void __launch_bounds__(1024) post_layer_norm_kernel(PostArgs a) {
   const T *post_w = static_cast<const T*>(a.post_w), *next_w = static_cast<const T*>(a.next_w);
   float* xr = a.x + t * W;
   float x[PER * 4], v[PER * 4], u[PER * 4];
+  pdl_trigger();
+  pdl_wait();
   // every load of the row is in flight before the first reduction
   if (!a.replace) {
     Share::load(xr, W, x);
@@ -161,6 +163,8 @@ __global__ void embed_bigram_kernel(const T* __restrict__ table, const T* __rest
                                     const int32_t* __restrict__ slot, const int32_t* __restrict__ pos, const int32_t* __restrict__ back,
                                     const int32_t* __restrict__ ahead, float* __restrict__ x, T* __restrict__ out) {
   __shared__ int64_t shared_row;
+  pdl_trigger();
+  pdl_wait();
   const int64_t t = blockIdx.x, token = tok[t];
   if (bigram) {
     if (threadIdx.x == 0) {
@@ -210,12 +214,12 @@ int launch_post(const PostArgs& a, int64_t n, cudaStream_t st) {
   int64_t th = ((groups + spread - 1) / spread + 31) / 32 * 32;
   th = th < 32 ? 32 : th > 1024 ? 1024 : th;
   const int64_t per = (groups + th - 1) / th;
-  if (per <= 1) post_layer_norm_kernel<T, 1, VEC><<<(unsigned)n, (unsigned)th, 0, st>>>(a);
-  else if (per <= 2) post_layer_norm_kernel<T, 2, VEC><<<(unsigned)n, (unsigned)th, 0, st>>>(a);
-  else if (per <= 4) post_layer_norm_kernel<T, 4, VEC><<<(unsigned)n, (unsigned)th, 0, st>>>(a);
-  else if (per <= 8) post_layer_norm_kernel<T, 8, VEC><<<(unsigned)n, (unsigned)th, 0, st>>>(a);
-  else return AO_B200_ERR_UNSUPPORTED;
-  return lm_launch_status();
+  const dim3 grid((unsigned)n), block((unsigned)th);
+  if (per <= 1) return lm_launch_early(post_layer_norm_kernel<T, 1, VEC>, grid, block, 0, st, a);
+  if (per <= 2) return lm_launch_early(post_layer_norm_kernel<T, 2, VEC>, grid, block, 0, st, a);
+  if (per <= 4) return lm_launch_early(post_layer_norm_kernel<T, 4, VEC>, grid, block, 0, st, a);
+  if (per <= 8) return lm_launch_early(post_layer_norm_kernel<T, 8, VEC>, grid, block, 0, st, a);
+  return AO_B200_ERR_UNSUPPORTED;
 }
 
 }  // namespace
@@ -245,8 +249,8 @@ extern "C" int ao_lm_embed_bigram(const void* table, const void* bigram, int dt,
   LM_DISPATCH(dt, {
     const bool vec = width % 4 == 0 && on(table, 4 * sizeof(T)) && on(bigram, 4 * sizeof(T)) && on(x, 16) && on(out, 4 * sizeof(T));
     auto kern = vec ? embed_bigram_kernel<T, true> : embed_bigram_kernel<T, false>;
-    kern<<<(unsigned)n, th, 0, lm_stream(stream)>>>(static_cast<const T*>(table), static_cast<const T*>(bigram), tok, width, scale, buckets,
-                                                     mul_prev, mul_cur, last, slot, pos, back, ahead, x, static_cast<T*>(out));
+    return lm_launch_early(kern, dim3((unsigned)n), dim3(th), 0, lm_stream(stream), static_cast<const T*>(table), static_cast<const T*>(bigram),
+                           tok, width, scale, buckets, mul_prev, mul_cur, last, slot, pos, back, ahead, x, static_cast<T*>(out));
   });
-  return lm_launch_status();
+  return AO_B200_OK;
 }

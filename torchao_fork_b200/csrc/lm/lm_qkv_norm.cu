@@ -32,6 +32,8 @@ __global__ void __launch_bounds__(kWarps * 32) qkv_norm_rotary_kernel(QkvArgs a)
   float *cs = sm, *sn = sm + hp;                                    // cosines and sines of the row's pairs
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* buf = sm + 2 * hp + (size_t)warp * dp;                     // this warp's head, normed
+  pdl_trigger();
+  pdl_wait();
   const int64_t t = blockIdx.x;
   const int p = a.pos[t];
   const float* row = a.proj + t * a.ld;
@@ -163,7 +165,7 @@ extern "C" int ao_lm_qkv_norm_rotary_prep(const float* proj, int64_t ld, int64_t
                      k_off % 4 == 0 && v_off % 4 == 0 && on(proj, 16) && on(qn, 16) && on(kn, four) && on(vn, four) && on(ring_k, four) &&
                      on(ring_v, four) && on(q_bias, four) && on(k_bias, four) && on(v_bias, four) && on(q_weight, four) && on(k_weight, four);
     auto kern = vec ? qkv_norm_rotary_kernel<T, true> : qkv_norm_rotary_kernel<T, false>;
-    kern<<<dim3((unsigned)n, parts), kWarps * 32, smem, lm_stream(stream)>>>(a);
+    return lm_launch_early(kern, dim3((unsigned)n, parts), dim3(kWarps * 32), smem, lm_stream(stream), a);
   });
-  return lm_launch_status();
+  return AO_B200_OK;
 }

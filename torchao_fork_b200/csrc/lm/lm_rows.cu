@@ -259,19 +259,29 @@ __global__ void add_cast_kernel(const T* __restrict__ b, int64_t count, float* _
 __global__ void argmax_kernel(const float* __restrict__ logits, int64_t ld, int64_t V, int64_t* __restrict__ out) {
   __shared__ float bv[32];
   __shared__ int64_t bi[32];
+  pdl_trigger();
+  pdl_wait();
   const float* row = logits + blockIdx.x * ld;
   float best = -INFINITY;
   int64_t at = V;
-  int64_t i = threadIdx.x;
-  for (; i + 3 * (int64_t)blockDim.x < V; i += 4 * (int64_t)blockDim.x) {   // four loads in flight per thread
-    float v[4];
+  int64_t done = 0;
+  if (ld % 4 == 0 && reinterpret_cast<uintptr_t>(logits) % 16 == 0) {
+    const int64_t groups = V / 4, step = blockDim.x;
+    for (int64_t i = threadIdx.x; i < groups; i += 8 * step) {   // eight 16-byte loads in flight per thread
+      float4 v[8];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) v[j] = row[i + j * (int64_t)blockDim.x];
+      for (int j = 0; j < 8; ++j) v[j] = i + j * step < groups ? ld4(row + (i + j * step) * 4) : make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
-      if (v[j] > best) best = v[j], at = i + j * (int64_t)blockDim.x;     // ascending indices: the first of equals stays
+      for (int j = 0; j < 8; ++j) {
+        const float f[4] = {v[j].x, v[j].y, v[j].z, v[j].w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (f[e] > best) best = f[e], at = (i + j * step) * 4 + e;     // ascending indices: the first of equals stays
+      }
+    }
+    done = groups * 4;
   }
-  for (; i < V; i += blockDim.x) {
+  for (int64_t i = done + threadIdx.x; i < V; i += blockDim.x) {
     const float v = row[i];
     if (v > best) best = v, at = i;
   }
@@ -411,6 +421,5 @@ extern "C" int ao_lm_add_cast(const void* b, int dt, int64_t count, float* a_ino
 
 extern "C" int ao_lm_argmax(const float* logits, int64_t ld, int64_t B, int64_t V, int64_t* out, void* stream) {
   LM_CHECK_ARG(logits && out && B > 0 && V > 0 && ld >= V);
-  argmax_kernel<<<(unsigned)B, 1024, 0, lm_stream(stream)>>>(logits, ld, V, out);
-  return lm_launch_status();
+  return lm_launch_early(argmax_kernel, dim3((unsigned)B), dim3(1024), 0, lm_stream(stream), logits, ld, V, out);
 }

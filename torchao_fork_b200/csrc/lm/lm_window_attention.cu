@@ -168,6 +168,8 @@ __device__ __forceinline__ void stage_key_block(float* dst, int stride, int widt
 template <typename T, int NM>
 __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WinArgs a) {
   extern __shared__ float sm[];
+  pdl_trigger();
+  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tile = blockIdx.x;
   const int d = a.d, dv = a.dv, G = a.G;
@@ -335,6 +337,8 @@ __global__ void __launch_bounds__(kWarps * 32) window_attention_kernel(WinArgs a
 template <typename T, int NM>
 __global__ void __launch_bounds__(kWarps * 32) window_attention_merge_kernel(WinArgs a) {
   extern __shared__ float sm[];    // [kWarps][NM][dv + 2], then [NM][dv]
+  pdl_trigger();
+  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tile = blockIdx.x, pr = blockIdx.z;
   const int dv = a.dv;
@@ -427,12 +431,10 @@ int launch_window(const WinArgs& a, int n_tiles, size_t smem, cudaStream_t st) {
     }
   }
   const unsigned gy = (unsigned)(a.G * win_head_shares(a.H, a.G));
-  kern<<<dim3((unsigned)n_tiles, gy, (unsigned)a.n_split), kWarps * 32, smem, st>>>(a);
-  if (a.n_split > 1) {
-    const size_t msm = ((size_t)kWarps * NM * (a.dv + 2) + (size_t)NM * a.dv) * sizeof(float);      // <= 19 KB
-    window_attention_merge_kernel<T, NM><<<dim3((unsigned)n_tiles, gy, kPairs), kWarps * 32, msm, st>>>(a);
-  }
-  return lm_launch_status();
+  const int rc = lm_launch_early(kern, dim3((unsigned)n_tiles, gy, (unsigned)a.n_split), dim3(kWarps * 32), smem, st, a);
+  if (rc != AO_B200_OK || a.n_split == 1) return rc;
+  const size_t msm = ((size_t)kWarps * NM * (a.dv + 2) + (size_t)NM * a.dv) * sizeof(float);      // <= 19 KB
+  return lm_launch_early(window_attention_merge_kernel<T, NM>, dim3((unsigned)n_tiles, gy, kPairs), dim3(kWarps * 32), msm, st, a);
 }
 
 }  // namespace
