@@ -71,6 +71,10 @@ class SozanexBench(Bench):
         heads = row.as_strided((H, 1, dv), (dv, H * dv, 1))
         ms = timed(lambda: torch.bmm(olat.transpose(0, 1), uv.transpose(1, 2), out=heads), flush=self.flush)
         self.bytes_row("batched_product_without_gate_decode", ms, uv.numel() * 2)
+        q1, qr0 = self.f32(1, H, dn + dr), self.f32(1, H, dr)
+        uk = self.bf(H, dn, R)
+        ms = self.call("latent_query_fold", q1, uk, BF16, 1, H, dn, dr, R, a.rot.dims, a.rot.inv_freq(self.dev), 1.1, self.last, qa, qr0)
+        self.bytes_row("latent_query_fold_decode", ms, uk.numel() * 2)
         # row kernels around it
         wq, wc, inv = self.bf(Rq), self.bf(R), a.rot.inv_freq(self.dev)
         cq, c, krr, cc, ck = self.bf(n, Rq), self.bf(n, R), self.bf(n, dr), self.bf(1, n, R), self.bf(1, n, dr)
@@ -143,12 +147,24 @@ class SozanexBench(Bench):
         ms = self.call("xielu_rows", f, ff, n, ff, 0.7, 1.1, ya, ff, BF16)
         self.bytes_row("rigalorn_xielu_rows", ms, n * ff * 6)
 
+    # ------------------------------------------------------------------------------------------------ products of one row
+    def products(self):
+        W, ff = self.W, self.ff
+        for key, M, K, act in (("up", ff, W, 1), ("down", W, ff, 0), ("o", W, W, 0), ("head", self.cfg.vocab_size, W, 0)):
+            x, w = self.bf(1, K), self.bf(M, K)
+            out = self.bf(1, M) if act else self.f32(1, M)
+            ms = self.call("gemv_rows", x, K, w, K, 1, M, K, act, out, M)
+            self.bytes_row(f"gemv_rows_{key}_one_row", ms, M * K * 2)
+            ms = timed(lambda: torch.mm(x, w.t(), out_dtype=torch.float32), flush=self.flush)
+            self.bytes_row(f"library_product_{key}_one_row", ms, M * K * 2)
+
 
 def kernel_numbers(name, prompt_len, decode_ctx):
     b = SozanexBench(name, prompt_len, decode_ctx)
     b.latent()
     b.attention()
     b.rows()
+    b.products()
     return b.res
 
 

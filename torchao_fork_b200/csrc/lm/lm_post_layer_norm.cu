@@ -13,36 +13,14 @@ namespace {
 
 constexpr int kMaxWarps = 32;
 
-// Mean and sum of squared deviations of a group of values; two groups merge exactly (up to rounding) without going back to
-// the values, so a row's variance needs ONE reduction instead of one for the mean and one for the deviations.
-struct Moments {
-  float n, mean, m2;
-};
-__device__ __forceinline__ Moments merged(const Moments& a, const Moments& b) {
-  const float n = a.n + b.n;
-  if (n == 0.f) return a;
-  const float d = b.mean - a.mean, share = b.n / n;
-  return {n, fmaf(d, share, a.mean), a.m2 + b.m2 + d * d * a.n * share};
-}
-__device__ __forceinline__ Moments warp_moments(Moments v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    Moments w;
-    w.n = __shfl_xor_sync(0xffffffffu, v.n, o);
-    w.mean = __shfl_xor_sync(0xffffffffu, v.mean, o);
-    w.m2 = __shfl_xor_sync(0xffffffffu, v.m2, o);
-    v = merged(v, w);
-  }
-  return v;
-}
-// over the block; every thread gets the result.  scratch: a buffer of its own per call in one kernel (one barrier per call).
-__device__ __forceinline__ Moments block_moments(Moments v, Moments* scratch) {
+// Sum over the block; every thread gets it.  scratch: kMaxWarps floats that no other sum of the kernel uses (one barrier per sum).
+__device__ __forceinline__ float block_total(float v, float* scratch) {
   const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  v = warp_moments(v);
+  v = warp_sum(v);
   if (nw == 1) return v;
   if (lane == 0) scratch[w] = v;
   __syncthreads();
-  return warp_moments(lane < nw ? scratch[lane] : Moments{0.f, 0.f, 0.f});
+  return warp_sum(lane < nw ? scratch[lane] : 0.f);
 }
 
 // A thread's share of a row: PER groups of four values.  VEC: group j is the four neighbours at 4 (threadIdx + j blockDim);
@@ -80,17 +58,20 @@ struct RowShare {
       }
     }
   }
-  static __device__ __forceinline__ Moments moments(int64_t W, const float (&v)[PER * 4]) {
-    float n = 0.f, s = 0.f;
+  // v = (v - mean) / sqrt(mean squared deviation + eps) * g; scratch: two sums' worth
+  static __device__ __forceinline__ void norm(int64_t W, float eps, const float (&g)[PER * 4], float (&v)[PER * 4], float (*scratch)[kMaxWarps]) {
+    float s = 0.f, ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < PER * 4; ++i)
-      if (at(i / 4, i % 4) < W) n += 1.f, s += v[i];
-    const float mean = n > 0.f ? s / n : 0.f;
-    float m2 = 0.f;
+    for (int i = 0; i < PER * 4; ++i) s += v[i];             // places past the row hold zeros
+    const float mean = block_total(s, scratch[0]) / (float)W;
 #pragma unroll
-    for (int i = 0; i < PER * 4; ++i)
-      if (at(i / 4, i % 4) < W) m2 = fmaf(v[i] - mean, v[i] - mean, m2);
-    return {n, mean, m2};
+    for (int i = 0; i < PER * 4; ++i) {
+      v[i] = at(i / 4, i % 4) < W ? v[i] - mean : 0.f;
+      ss = fmaf(v[i], v[i], ss);
+    }
+    const float k = 1.f / sqrtf(block_total(ss, scratch[1]) / (float)W + eps);
+#pragma unroll
+    for (int i = 0; i < PER * 4; ++i) v[i] *= k * g[i];
   }
 };
 
@@ -107,7 +88,7 @@ struct PostArgs {
 template <typename T, int PER, bool VEC>
 __global__ void __launch_bounds__(1024) post_layer_norm_kernel(PostArgs a) {
   using Share = RowShare<PER, VEC>;
-  __shared__ Moments scratch[2][kMaxWarps];
+  __shared__ float scratch[4][kMaxWarps];
   const int64_t t = blockIdx.x, W = a.W;
   const T *post_w = static_cast<const T*>(a.post_w), *next_w = static_cast<const T*>(a.next_w);
   float* xr = a.x + t * W;
@@ -130,14 +111,10 @@ __global__ void __launch_bounds__(1024) post_layer_norm_kernel(PostArgs a) {
     }
     if (post_w) {
       Share::load(post_w, W, u);
-      const Moments m = block_moments(Share::moments(W, v), scratch[0]);
-      const float k = 1.f / sqrtf(m.m2 / (float)W + a.eps);
-#pragma unroll
-      for (int i = 0; i < PER * 4; ++i) x[i] = fmaf((v[i] - m.mean) * k, u[i], x[i]);
-    } else {
-#pragma unroll
-      for (int i = 0; i < PER * 4; ++i) x[i] += v[i];
+      Share::norm(W, a.eps, u, v, scratch);
     }
+#pragma unroll
+    for (int i = 0; i < PER * 4; ++i) x[i] += v[i];
     if (a.add_rows) {
       Share::load(a.add_rows + t * a.ld_add, W, v);
 #pragma unroll
@@ -149,10 +126,7 @@ __global__ void __launch_bounds__(1024) post_layer_norm_kernel(PostArgs a) {
   T* out = static_cast<T*>(a.out) + t * a.ld_out;
   if (next_w) {
     Share::load(next_w, W, u);
-    const Moments m = block_moments(Share::moments(W, x), scratch[1]);
-    const float k = 1.f / sqrtf(m.m2 / (float)W + a.eps);
-#pragma unroll
-    for (int i = 0; i < PER * 4; ++i) x[i] = (x[i] - m.mean) * k * u[i];
+    Share::norm(W, a.eps, u, x, scratch + 2);
   }
   Share::store(out, W, x);
 }
