@@ -132,6 +132,8 @@ class SozanexBench(Bench):
         self.bytes_row("rigalorn_add_rms_norm", ms, n * W * 14)
         ms = self.call("add_layer_norm", x, None, 0.0, None, n, W, w, None, BF16, 1e-6, None, h)
         self.bytes_row("final_layer_norm", ms, n * W * 6)
+        ms = self.call("add_rms_norm", x, None, None, n, W, w, BF16, 1e-6, h)
+        self.bytes_row("rigalorn_final_rms_norm", ms, n * W * 6)
         b = self.cfg.bigram
         table, big = self.bf(self.cfg.vocab_size, W), self.bf(b.buckets + 1, W)
         tok = torch.randint(0, self.cfg.vocab_size, (n,), device=self.dev)
